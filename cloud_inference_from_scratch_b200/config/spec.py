@@ -131,6 +131,9 @@ class ModelSpec:
     # every sublayer's result is multiplied by this constant as it is added to the stream (the norms of such a
     # model are built with the same constant as their ``update_scale``)
     residual_scale: float = 1.0
+    # a norm that the embedding rows pass before the first layer (None: none)
+    embedding_norm: PartSpec | None = None
+    embedding_norm_prefix: str = ""
 
     def validate(self) -> None:
         if not self.layers:
@@ -139,6 +142,8 @@ class ModelSpec:
             raise ValueError("logit_softcap must be >= 0")
         if self.residual_streams < 1:
             raise ValueError("residual_streams must be >= 1")
+        if self.embedding_norm is not None and self.residual_streams != 1:
+            raise ValueError("a norm on the embedding rows is built for one residual stream")
         if self.position_wave_base is not None and not self.position_wave_base > 0:
             raise ValueError("position_wave_base must be positive")
         rows_of = dict(self.offset_tensors)

@@ -19,6 +19,10 @@
 //
 // `sinks` != nullptr: the softmax denominator of query head h holds one more term exp(sinks[h]), which has no
 // key and no value and is not scaled.
+//
+// `cap` > 0: the scaled score becomes cap * tanh(score / cap).  `slopes` != nullptr: after that the score of a key at
+// position j is lowered by slopes[h] * (p - j).  `gates` != nullptr: head h's output is multiplied by
+// sigmoid(gates[t * gate_stride + h]) as it is written.
 #include "common.cuh"
 
 #include <cfloat>
@@ -30,6 +34,21 @@ namespace cie {
 constexpr int kMaxDim = 256;
 constexpr int kWarps = 4;
 
+// What lies around the plain score and output: see the head of this file (every pointer may be null).
+struct Options {
+  const float* r1;
+  const float* r2;
+  const float* sinks;
+  const float* slopes;
+  const float* gates;
+  int gate_stride;
+  float cap;
+};
+
+__device__ __forceinline__ float head_gate(const Options& o, int t, int h) {
+  return o.gates ? 1.f / (1.f + expf(-o.gates[(size_t)t * o.gate_stride + h])) : 1.f;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kWarps * 32)
 attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out, int out_stride,
@@ -37,8 +56,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
                          const int* __restrict__ positions, const int* __restrict__ request_of_token,
                          const int* __restrict__ table, int table_width, int num_pages, int tokens,
                          int q_heads, int kv_heads, int dim, int vdim, int page_size, float scale, int window,
-                         int keep_first, const float* __restrict__ r1, const float* __restrict__ r2,
-                         const float* __restrict__ sinks, int* err) {
+                         int keep_first, const Options opt, int* err) {
   __shared__ float q_s[kWarps][kMaxDim];
   __shared__ float p_s[kWarps][32];
   __shared__ long long off_s[kWarps][32];
@@ -58,7 +76,9 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
   if (first > keep_first) kept = keep_first;
   else first = 0;
   const int visible = kept + length - first;
-  const float penalty = r1 ? r1[h] : 0.f, reach = r1 ? r2[h] : 0.f;
+  const float *r1 = opt.r1, *sinks = opt.sinks;
+  const float penalty = r1 ? r1[h] : 0.f, reach = r1 ? opt.r2[h] : 0.f;
+  const float slope = opt.slopes ? opt.slopes[h] : 0.f;
 
   const T* qv = q + (size_t)t * q_stride + (size_t)h * dim;
   for (int d = lane; d < dim; d += 32) q_s[warp][d] = to_float(qv[d]);
@@ -89,7 +109,9 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
       float dot = 0.f;
       for (int d = 0; d < dim; ++d) dot = fmaf(q_s[warp][d], to_float(kr[d]), dot);
       s = dot * scale;
+      if (opt.cap > 0.f) s = opt.cap * tanhf(s / opt.cap);
       if (r1) s -= penalty * log1pf(reach * (float)(pos - key));
+      s -= slope * (float)(pos - key);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float p = offset >= 0 ? expf(s - m_new) : 0.f;
@@ -122,7 +144,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
     keep = expf(m - top);
     l = l * keep + expf(sinks[h] - top);
   }
-  const float inv = l > 0.f ? keep / l : 0.f;
+  const float inv = (l > 0.f ? keep / l : 0.f) * head_gate(opt, t, h);
 #pragma unroll
   for (int i = 0; i < kMaxDim / 32; ++i) {
     const int d = lane + 32 * i;
@@ -162,8 +184,7 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
                        const int* __restrict__ positions, const int* __restrict__ request_of_token,
                        const int* __restrict__ table, int table_width, int num_pages, int q_heads,
                        int kv_heads, int dim, int vdim, int page_size, float scale, int window, int keep_first,
-                       const float* __restrict__ r1, const float* __restrict__ r2,
-                       const float* __restrict__ sinks, int splits,
+                       const Options opt, int splits,
                        float* __restrict__ shares, int* __restrict__ tickets, int* err) {
   // splits > 1: the keys of a token are cut into that many ranges, one CTA each (blockIdx.x = token *
   // splits + range); a CTA leaves its maximum, sum and unnormalised output in `shares`, and whoever
@@ -199,11 +220,13 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
     const int h = e / dim, d = e % dim;
     q_s[e] = h < heads ? to_float(q[(size_t)t * q_stride + (size_t)(kvh * group + h0 + h) * dim + d]) : 0.f;
   }
-  float penalty[kGroupHeads], reach[kGroupHeads];
+  const float *r1 = opt.r1, *sinks = opt.sinks;
+  float penalty[kGroupHeads], reach[kGroupHeads], slope[kGroupHeads];
 #pragma unroll
   for (int h = 0; h < kGroupHeads; ++h) {
     penalty[h] = (r1 && h < heads) ? r1[kvh * group + h0 + h] : 0.f;
-    reach[h] = (r1 && h < heads) ? r2[kvh * group + h0 + h] : 0.f;
+    reach[h] = (r1 && h < heads) ? opt.r2[kvh * group + h0 + h] : 0.f;
+    slope[h] = (opt.slopes && h < heads) ? opt.slopes[kvh * group + h0 + h] : 0.f;
   }
   __syncthreads();
   float m[kGroupHeads], l[kGroupHeads], acc[kGroupHeads][kGroupMaxV / 32];
@@ -258,7 +281,9 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
       float s = -FLT_MAX;
       if (slot >= 0) {
         s = dot[h] * scale;
+        if (opt.cap > 0.f) s = opt.cap * tanhf(s / opt.cap);
         if (r1) s -= penalty[h] * log1pf(reach[h] * distance);
+        s -= slope[h] * distance;
       }
       const float m_new = fmaxf(m[h], warp_max(s));
       const float p = slot >= 0 ? expf(s - m_new) : 0.f;
@@ -317,7 +342,8 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
       value = fmaf(share, o_s[(w * kGroupHeads + h) * kGroupMaxV + d], value);
     }
     if (splits == 1) {
-      out[(size_t)t * out_stride + (size_t)(kvh * group + h0 + h) * vdim + d] = from_float<T>(sum > 0.f ? value / sum : 0.f);
+      out[(size_t)t * out_stride + (size_t)(kvh * group + h0 + h) * vdim + d] =
+        from_float<T>((sum > 0.f ? value / sum : 0.f) * head_gate(opt, t, kvh * group + h0 + h));
     } else {
       my_share[h * kShare + d] = value;
       if (d == 0) {
@@ -351,7 +377,8 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
       sum = fmaf(share, __ldcg(part + kGroupMaxV + 1), sum);
       value = fmaf(share, __ldcg(part + d), value);
     }
-    out[(size_t)t * out_stride + (size_t)(kvh * group + h0 + h) * vdim + d] = from_float<T>(sum > 0.f ? value / sum : 0.f);
+    out[(size_t)t * out_stride + (size_t)(kvh * group + h0 + h) * vdim + d] =
+        from_float<T>((sum > 0.f ? value / sum : 0.f) * head_gate(opt, t, kvh * group + h0 + h));
   }
 }
 
@@ -367,16 +394,19 @@ extern "C" int cie_attention_group_share_floats() { return kGroupHeads * (kGroup
 // keys are cut into that many ranges with a CTA each; `shares` holds tokens * kv_heads *
 // ceil(group / 8) * splits * cie_attention_group_share_floats() floats and `tickets` one int, zero, per
 // (token, kv head, 8 heads).
-// sinks: float32 [q_heads] or nullptr.
+// sinks: float32 [q_heads] or nullptr.  slopes, cap, gates (rows of gate_stride floats): see the head of this file.
 extern "C" int cie_attention_generic_sink(const void* q, int q_stride, void* out, int out_stride,
                                           const void* k_pool, const void* v_pool, const int* positions,
                                           const int* request_of_token, const int* table, int table_width,
                                           int num_pages, int tokens, int q_heads, int kv_heads, int dim,
                                           int vdim, int page_size, float scale, int window,
                                           const float* r1, const float* r2, int splits, float* shares,
-                                          int* tickets, int keep_first, const float* sinks, int dtype, int* err,
+                                          int* tickets, int keep_first, const float* sinks, const float* slopes,
+                                          float cap, const float* gates, int gate_stride, int dtype, int* err,
                                           void* stream) {
   if (tokens <= 0) return 0;
+  if (cap < 0.f) CIE_FAIL("attention_generic: a cap of %f", cap);
+  const Options opt{r1, r2, sinks, slopes, gates, gate_stride, cap};
   if (keep_first < 0) CIE_FAIL("attention_generic: %d kept keys", keep_first);
   if (splits < 1 || (splits > 1 && (!shares || !tickets))) CIE_FAIL("attention_generic: %d key ranges need shares and tickets", splits);
   if (dim > kMaxDim || dim < 1 || vdim > kMaxDim || vdim < 1)
@@ -407,7 +437,7 @@ extern "C" int cie_attention_generic_sink(const void* q, int q_stride, void* out
     CIE_LAUNCH("attention_group", (attention_group_kernel<T, S>), grid, dim3(kGroupWarps * 32), smem, s,            \
                (const T*)q, q_stride, (T*)out, out_stride, (const T*)k_pool, (const T*)v_pool, positions,          \
                request_of_token, table, table_width, num_pages, q_heads, kv_heads, dim, vdim, page_size, scale,    \
-               window, keep_first, r1, r2, sinks, splits, shares, tickets, err);                                   \
+               window, keep_first, opt, splits, shares, tickets, err);                                   \
   } while (0)
     if (dtype == kFloat32) CIE_GROUP(float, false);
     else if (staged) CIE_GROUP(__nv_bfloat16, true);
@@ -419,12 +449,12 @@ extern "C" int cie_attention_generic_sink(const void* q, int q_stride, void* out
     CIE_LAUNCH("attention_generic", attention_generic_kernel<float>, dim3(blocks), dim3(kWarps * 32), 0, s,
         (const float*)q, q_stride, (float*)out, out_stride, (const float*)k_pool, (const float*)v_pool,
         positions, request_of_token, table, table_width, num_pages, tokens, q_heads, kv_heads, dim, vdim,
-        page_size, scale, window, keep_first, r1, r2, sinks, err);
+        page_size, scale, window, keep_first, opt, err);
   } else if (dtype == kBFloat16) {
     CIE_LAUNCH("attention_generic", attention_generic_kernel<__nv_bfloat16>, dim3(blocks), dim3(kWarps * 32), 0, s,
         (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_pool,
         (const __nv_bfloat16*)v_pool, positions, request_of_token, table, table_width, num_pages, tokens,
-        q_heads, kv_heads, dim, vdim, page_size, scale, window, keep_first, r1, r2, sinks, err);
+        q_heads, kv_heads, dim, vdim, page_size, scale, window, keep_first, opt, err);
   } else {
     CIE_FAIL("attention_generic: unknown element type code %d", dtype);
   }

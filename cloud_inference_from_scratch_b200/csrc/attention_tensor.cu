@@ -38,6 +38,7 @@ namespace cg = cooperative_groups;
 // (fragment loads, tile addressing, score / accumulate / softmax steps: attention_tiles.cuh)
 // ------------------------------------------------------------------------------------ prefill
 constexpr int BM = 128, BN = 64, PREFILL_WARPS = 8;
+constexpr float kLog2eF = 1.4426950408889634f;
 
 struct PrefillArgs {
   const bf16* q;
@@ -66,6 +67,15 @@ struct PrefillArgs {
   // one more term exp(sinks[h]) in the softmax denominator of query head h (no key, no value, not scaled);
   // nullptr: none
   const float* sinks;
+  // key and value elements of a head in use (multiples of 16 up to the build's head size)
+  int kdim, vdim;
+  // the scaled score becomes cap * tanh(score / cap) (0: no cap), and is then lowered by slopes[h] * (position - key)
+  // (nullptr: not)
+  float cap;
+  const float* slopes;
+  // head h of token t is multiplied by sigmoid(gates[t * gate_stride + h]) as it is written (nullptr: not)
+  const float* gates;
+  int gate_stride;
 };
 
 // One 64-key tile: thread t < 64 copies key row t of K, thread 64 + t row t of V, each with one bulk
@@ -78,20 +88,23 @@ __device__ __forceinline__ int kv_tile_rows(int k0, int valid_lo, int valid_hi, 
 
 __device__ __forceinline__ void load_kv_tile(const PrefillArgs& a, const int* row, int kvh, int k0,
                                              int valid_lo, int valid_hi, int kept, bf16* k_dst, bf16* v_dst,
-                                             uint64_t* bar, int tid) {
+                                             uint64_t* bar, int tid, int kdim, int vdim) {
   const int rows = kv_tile_rows(k0, valid_lo, valid_hi, kept);
-  if (tid == 0) mbar_expect_tx(bar, (uint32_t)rows * 2u * ROW_BYTES);
+  if (tid == 0) mbar_expect_tx(bar, (uint32_t)rows * (uint32_t)(kdim + vdim) * 2u);
   if (tid >= 2 * BN) return;
   const int r = tid & (BN - 1);
   const int key = k0 + r;
   if (key >= valid_hi || (key < valid_lo && key >= kept)) return;
-  long long off = kv_offset(a.pools, row, key, kvh, a.err);
-  if (off < 0) off = (long long)kvh * a.pools.page_size * D;   // page 0: the copy must still happen
-  if (tid < BN) bulk_copy(k_dst + r * ROW, a.pools.k + off, ROW_BYTES, bar);
-  else bulk_copy(v_dst + r * ROW, a.pools.v + off, ROW_BYTES, bar);
+  long long at = kv_row(a.pools, row, key, kvh, a.err);
+  if (at < 0) at = (long long)kvh * a.pools.page_size;   // page 0: the copy must still happen
+  if (tid < BN) bulk_copy(k_dst + r * ROW, a.pools.k + at * kdim, (uint32_t)kdim * 2u, bar);
+  else bulk_copy(v_dst + r * ROW, a.pools.v + at * vdim, (uint32_t)vdim * 2u, bar);
 }
 
+// kFull: key and value heads have the build's size.
+template <bool kFull>
 __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const PrefillArgs a) {
+  const int kdim = kFull ? D : a.kdim, vdim = kFull ? D : a.vdim;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);  // [BM][ROW]
   bf16* k_s = q_s + BM * ROW;                     // [2][BN][ROW]
@@ -111,8 +124,8 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const Prefi
   for (int idx = tid; idx < BM * CHUNKS; idx += PREFILL_WARPS * 32) {
     const int r = idx / CHUNKS, c = idx % CHUNKS;
     const int tok = r / a.hpt, hh = h0 + r % a.hpt;
-    const bool ok = tok < ntok && hh < a.group;
-    const bf16* src = ok ? a.q + (size_t)(first_token + tok) * a.q_stride + (size_t)(kvh * a.group + hh) * D + c * 8 : a.q;
+    const bool ok = tok < ntok && hh < a.group && c * 8 < kdim;
+    const bf16* src = ok ? a.q + (size_t)(first_token + tok) * a.q_stride + (size_t)(kvh * a.group + hh) * kdim + c * 8 : a.q;
     cp_async16(q_s + r * ROW + c * 8, src, ok);
   }
   cp_async_commit();
@@ -132,7 +145,7 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const Prefi
   if (tid < 2) mbar_init(&bars[tid], 1);
   asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   __syncthreads();
-  load_kv_tile(a, table_row, kvh, tile_k0(0), valid_lo, valid_hi, kept, k_s, v_s, &bars[0], tid);
+  load_kv_tile(a, table_row, kvh, tile_k0(0), valid_lo, valid_hi, kept, k_s, v_s, &bars[0], tid, kdim, vdim);
 
   uint32_t q_frag[KSTEPS][4];
   float o[NTILES_D][4];
@@ -143,7 +156,9 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const Prefi
   // positions of the two rows this thread holds (-1: row not in use)
   const int g = lane >> 2, t4 = lane & 3;
   int row_pos[2];
-  float row_r1[2] = {0.f, 0.f}, row_r2[2] = {0.f, 0.f};
+  float row_r1[2] = {0.f, 0.f}, row_r2[2] = {0.f, 0.f}, row_slope[2] = {0.f, 0.f};
+  // cap * tanh(s / cap) = cap - 2 cap / (exp(2 s / cap) + 1), in units of log 2
+  const float cap_log2 = a.cap * kLog2eF, to_exponent = a.cap > 0.f ? 2.f * kLog2eF / cap_log2 : 0.f;
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int r = warp * 16 + g + h * 8;
@@ -153,6 +168,7 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const Prefi
       row_r1[h] = a.r1[kvh * a.group + hh];
       row_r2[h] = a.r2[kvh * a.group + hh];
     }
+    if (a.slopes && row_pos[h] >= 0) row_slope[h] = a.slopes[kvh * a.group + hh] * kLog2eF;
   }
 
   bool alive = true;
@@ -160,7 +176,7 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const Prefi
     const int stage = it & 1;
     if (it + 1 < tiles)
       load_kv_tile(a, table_row, kvh, tile_k0(it + 1), valid_lo, valid_hi, kept,
-                   k_s + (stage ^ 1) * BN * ROW, v_s + (stage ^ 1) * BN * ROW, &bars[stage ^ 1], tid);
+                   k_s + (stage ^ 1) * BN * ROW, v_s + (stage ^ 1) * BN * ROW, &bars[stage ^ 1], tid, kdim, vdim);
     if (it == 0) cp_async_wait<0>();   // the queries
     alive = mbar_wait(&bars[stage], (it >> 1) & 1, a.err);
     const int k0 = tile_k0(it);
@@ -187,7 +203,7 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const Prefi
     const int warp_pos_hi = context + q0 + min(ntok - 1, (warp * 16 + 15) / a.hpt);
     if (k0 <= warp_pos_hi) {
       float s[BN / 8][4];
-      scores<BN / 16>(q_frag, k_s + stage * BN * ROW, s, lane);
+      scores<BN / 16>(q_frag, k_s + stage * BN * ROW, s, lane, kdim / 16);
 #pragma unroll
       for (int i = 0; i < BN / 8; ++i) {
 #pragma unroll
@@ -196,13 +212,15 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const Prefi
           const int pos = row_pos[e >> 1];
           const bool ok = key <= pos && (a.window <= 0 || key > pos - a.window || key < a.keep_first);
           float score = s[i][e] * a.scale_log2;
+          if (a.cap > 0.f) score = fmaf(-2.f * cap_log2, __fdividef(1.f, exp2f(score * to_exponent) + 1.f), cap_log2);
+          score = fmaf(-row_slope[e >> 1], (float)(pos - key), score);
           if (a.r1 && ok) score -= row_r1[e >> 1] * __log2f(fmaf(row_r2[e >> 1], (float)(pos - key), 1.f));
           s[i][e] = ok ? score : -INFINITY;
         }
       }
       softmax_update<BN / 8>(s, m, l, o);
-      if (a.split_weights) accumulate_split<BN / 16>(s, v_s + stage * BN * ROW, o, lane);
-      else accumulate<BN / 16>(s, v_s + stage * BN * ROW, o, lane);
+      if (a.split_weights) accumulate_split<BN / 16>(s, v_s + stage * BN * ROW, o, lane, vdim / 16);
+      else accumulate<BN / 16>(s, v_s + stage * BN * ROW, o, lane, vdim / 16);
     }
     __syncthreads();
   }
@@ -221,10 +239,12 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32) prefill_kernel(const Prefi
       keep = exp2f(m[h] - top);
       total = total * keep + exp2f(sink - top);
     }
-    const float inv = total > 0.f ? keep / total : 0.f;
-    bf16* dst = a.out + (size_t)(first_token + tok) * a.out_stride + (size_t)(kvh * a.group + hh) * D;
+    float inv = total > 0.f ? keep / total : 0.f;
+    if (a.gates) inv /= 1.f + expf(-a.gates[(size_t)(first_token + tok) * a.gate_stride + kvh * a.group + hh]);
+    bf16* dst = a.out + (size_t)(first_token + tok) * a.out_stride + (size_t)(kvh * a.group + hh) * vdim;
 #pragma unroll
     for (int i = 0; i < NTILES_D; ++i) {
+      if (i * 8 >= vdim) break;
       const uint32_t packed = pack_bf16(o[i][2 * h] * inv, o[i][2 * h + 1] * inv);
       *reinterpret_cast<uint32_t*>(dst + i * 8 + 2 * t4) = packed;
     }
@@ -1156,7 +1176,8 @@ extern "C" int cie_attention_head_dim() { return D; }
 
 // r1, r2: float32 [q_heads] of the distance penalty, or both null; split_weights: 1 keeps the
 // softmax weights to 16 bits of mantissa in the value product (two bfloat16 terms); keep_first: with a window,
-// the request's first so many keys stay visible behind it; sinks: float32 [q_heads] or null.
+// the request's first so many keys stay visible behind it; sinks: float32 [q_heads] or null; kdim, vdim: key and
+// value elements of a head (multiples of 16 up to the build's head size); cap, slopes, gates: see PrefillArgs.
 extern "C" int cie_attention_prefill_ex(const void* q, int q_stride, void* out, int out_stride,
                                         const void* k_pool, const void* v_pool, const int* table,
                                         int table_width, int num_pages, const int* tile_request,
@@ -1164,8 +1185,12 @@ extern "C" int cie_attention_prefill_ex(const void* q, int q_stride, void* out, 
                                         const int* query_lens, const int* query_start, int q_heads,
                                         int kv_heads, int page_size, int hpt, float scale, int window,
                                         const float* r1, const float* r2, int split_weights, int keep_first,
-                                        const float* sinks, int* err, void* stream) {
+                                        const float* sinks, int kdim, int vdim, float cap, const float* slopes,
+                                        const float* gates, int gate_stride, int* err, void* stream) {
   if (num_tiles <= 0) return 0;
+  if (kdim < 16 || kdim > D || kdim % 16 || vdim < 16 || vdim > D || vdim % 16)
+    CIE_FAIL("attention_prefill: head sizes %d / %d are no multiples of 16 up to %d", kdim, vdim, D);
+  if (cap < 0.f) CIE_FAIL("attention_prefill: a cap of %f", cap);
   if (keep_first < 0) CIE_FAIL("attention_prefill: %d kept first keys", keep_first);
   if ((r1 == nullptr) != (r2 == nullptr)) CIE_FAIL("attention_prefill: the distance penalty needs both of its vectors");
   if (kv_heads < 1 || q_heads % kv_heads) CIE_FAIL("attention_prefill: %d query heads over %d kv heads", q_heads, kv_heads);
@@ -1180,15 +1205,21 @@ extern "C" int cie_attention_prefill_ex(const void* q, int q_stride, void* out, 
   a.group = group; a.hpt = hpt; a.tpt = BM / hpt; a.head_chunks = (group + hpt - 1) / hpt;
   a.scale_log2 = scale * kLog2e; a.window = window; a.keep_first = window > 0 ? keep_first : 0; a.err = err;
   a.r1 = r1; a.r2 = r2; a.split_weights = split_weights; a.sinks = sinks;
+  a.kdim = kdim; a.vdim = vdim; a.cap = cap; a.slopes = slopes; a.gates = gates; a.gate_stride = gate_stride;
   const size_t smem = (size_t)(BM + 4 * BN) * ROW * sizeof(bf16);
   static bool configured = false;
   if (!configured) {
-    cudaError_t status = cudaFuncSetAttribute(prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t status = cudaFuncSetAttribute(prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (status == cudaSuccess)
+      status = cudaFuncSetAttribute(prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (status != cudaSuccess) CIE_FAIL("attention_prefill: shared memory %zu: %s", smem, cudaGetErrorString(status));
     configured = true;
   }
   dim3 grid(num_tiles, kv_heads * a.head_chunks);
-  CIE_LAUNCH("attention_prefill", prefill_kernel, grid, dim3(PREFILL_WARPS * 32), smem, (cudaStream_t)stream, a);
+  if (kdim == D && vdim == D)
+    CIE_LAUNCH("attention_prefill", prefill_kernel<true>, grid, dim3(PREFILL_WARPS * 32), smem, (cudaStream_t)stream, a);
+  else
+    CIE_LAUNCH("attention_prefill", prefill_kernel<false>, grid, dim3(PREFILL_WARPS * 32), smem, (cudaStream_t)stream, a);
   return 0;
 }
 
@@ -1202,7 +1233,7 @@ extern "C" int cie_attention_prefill(const void* q, int q_stride, void* out, int
   return cie_attention_prefill_ex(q, q_stride, out, out_stride, k_pool, v_pool, table, table_width, num_pages,
                                   tile_request, tile_q0, num_tiles, context_lens, query_lens, query_start,
                                   q_heads, kv_heads, page_size, hpt, scale, window, nullptr, nullptr, 0, 0, nullptr,
-                                  err, stream);
+                                  D, D, 0.f, nullptr, nullptr, 0, err, stream);
 }
 
 // splits: CTAs that share the keys of one request (a thread-block cluster): 1, 2, 4 or 8.

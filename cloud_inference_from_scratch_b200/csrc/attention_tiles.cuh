@@ -78,20 +78,21 @@ struct Pools {
   int page_size;
 };
 
-// Address of key `key` of request row `row` for kv head `kvh`, or nullptr (and an error bit) if
+// Row of key `key` of request row `row` for kv head `kvh` in the pools, or -1 (and an error bit) if
 // the block table has no page there.
-__device__ __forceinline__ long long kv_offset(const Pools& pools, const int* row, int key, int kvh, int* err) {
+__device__ __forceinline__ long long kv_row(const Pools& pools, const int* row, int key, int kvh, int* err) {
   const int index = key / pools.page_size;
   const int page = index < pools.table_width ? row[index] : -1;
   if (page < 0 || page >= pools.num_pages) {
     atomicOr(err, kErrBadPage);
     return -1;
   }
-  return (((long long)page * pools.kv_heads + kvh) * pools.page_size + key % pools.page_size) * D;
+  return ((long long)page * pools.kv_heads + kvh) * pools.page_size + key % pools.page_size;
 }
 
 // One 16-row block against NB*16 keys held in shared memory (rows of ROW elements).
-// q_frag: A fragments of the 16 query rows.  s: NB*2 score tiles of 16 x 8.
+// q_frag: A fragments of the 16 query rows.  s: NB*2 score tiles of 16 x 8.  ksteps (below: dsteps): 16-element steps of
+// a head that are in use.
 // Address of element (row, col) of a key/value tile in shared memory, col a multiple of 8.
 // SW == false: rows of ROW elements (padded).  SW == true: the layout a TMA tensor copy with
 // 128-byte swizzle leaves: 16-row sub-tiles of 64 columns, 2 KB each, the 16-byte piece c of
@@ -109,7 +110,7 @@ __device__ __forceinline__ const bf16* tile_ptr(const bf16* base, int row, int c
 
 template <int NB, bool SW = false>
 __device__ __forceinline__ void scores(const uint32_t (&q_frag)[KSTEPS][4], const bf16* k_tile,
-                                       float (&s)[NB * 2][4], int lane) {
+                                       float (&s)[NB * 2][4], int lane, int ksteps = KSTEPS) {
   static_assert(!SW || NB == 1, "swizzled tiles hold 16 keys");
   // two accumulator sets (even and odd k-steps) halve the chain of dependent tensor-core
   // instructions; they are added at the end
@@ -122,6 +123,7 @@ __device__ __forceinline__ void scores(const uint32_t (&q_frag)[KSTEPS][4], cons
   const int mi = lane >> 3, r = lane & 7;
 #pragma unroll
   for (int kk = 0; kk < KSTEPS; ++kk) {
+    if (kk >= ksteps) break;
 #pragma unroll
     for (int nb = 0; nb < NB; ++nb) {
       uint32_t b[4];
@@ -144,7 +146,7 @@ __device__ __forceinline__ void scores(const uint32_t (&q_frag)[KSTEPS][4], cons
 // o += P V for NB*16 keys; p: probabilities in the score-tile layout.
 template <int NB, bool SW = false>
 __device__ __forceinline__ void accumulate(const float (&p)[NB * 2][4], const bf16* v_tile,
-                                           float (&o)[NTILES_D][4], int lane) {
+                                           float (&o)[NTILES_D][4], int lane, int dsteps = KSTEPS) {
   const int mi = lane >> 3, r = lane & 7;
 #pragma unroll
   for (int kb = 0; kb < NB; ++kb) {
@@ -155,6 +157,7 @@ __device__ __forceinline__ void accumulate(const float (&p)[NB * 2][4], const bf
     a[3] = pack_bf16(p[2 * kb + 1][2], p[2 * kb + 1][3]);
 #pragma unroll
     for (int db = 0; db < KSTEPS; ++db) {
+      if (db >= dsteps) break;
       uint32_t b[4];
       ldsm_x4_trans(b, tile_ptr<SW>(v_tile, kb * 16 + (mi & 1) * 8 + r, db * 16 + (mi >> 1) * 8));
       mma_bf16(o[2 * db], a, b[0], b[1]);
@@ -168,7 +171,7 @@ __device__ __forceinline__ void accumulate(const float (&p)[NB * 2][4], const bf
 // value product sees the weights to within 2^-17 of their size instead of 2^-9.
 template <int NB, bool SW = false>
 __device__ __forceinline__ void accumulate_split(const float (&p)[NB * 2][4], const bf16* v_tile,
-                                                 float (&o)[NTILES_D][4], int lane) {
+                                                 float (&o)[NTILES_D][4], int lane, int dsteps = KSTEPS) {
   const int mi = lane >> 3, r = lane & 7;
 #pragma unroll
   for (int kb = 0; kb < NB; ++kb) {
@@ -182,6 +185,7 @@ __device__ __forceinline__ void accumulate_split(const float (&p)[NB * 2][4], co
     }
 #pragma unroll
     for (int db = 0; db < KSTEPS; ++db) {
+      if (db >= dsteps) break;
       uint32_t b[4];
       ldsm_x4_trans(b, tile_ptr<SW>(v_tile, kb * 16 + (mi & 1) * 8 + r, db * 16 + (mi >> 1) * 8));
       mma_bf16(o[2 * db], hi, b[0], b[1]);

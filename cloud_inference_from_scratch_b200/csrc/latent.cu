@@ -42,7 +42,7 @@ latent_prepare_kernel(const float* __restrict__ down, int stride, T* __restrict_
                       const int* __restrict__ table, int table_width, int num_pages, T* __restrict__ c_pool,
                       T* __restrict__ r_pool, const float* __restrict__ inv_freq, float magnitude, int interleaved,
                       int rot_dims, int q_rank, int rank, int rot, int page_size, float eps, int has_kv,
-                      int write_cache, int* err) {
+                      int write_cache, const int* __restrict__ active, int* err) {
   __shared__ float scratch[33];
   pdl_wait();
   pdl_trigger();
@@ -56,6 +56,7 @@ latent_prepare_kernel(const float* __restrict__ down, int stride, T* __restrict_
       q_out[(size_t)t * q_rank + i] = from_float<T>(q_gain[i] * (row[i] * inv));
   }
   if (!has_kv || !write_cache) return;
+  if (active && !active[request_of_token[t]]) return;     // a row that only pads the batch
   const float* kv = row + q_rank;
   float sq = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) sq += kv[i] * kv[i];
@@ -427,7 +428,8 @@ extern "C" int cie_latent_prepare(const float* down, int stride, void* q_out, co
                                   const int* table, int table_width, int num_pages, void* c_pool, void* r_pool,
                                   const float* inv_freq, float magnitude, int interleaved, int rot_dims,
                                   int tokens, int q_rank, int rank, int rot, int page_size, float eps, int has_kv,
-                                  int write_cache, int dtype, int* err, void* stream) {
+                                  int write_cache, const int* active, int dtype, int* err, void* stream) {
+  // active: per request, 0 for a row that only pads the batch and writes nothing to the pages (nullptr: all write)
   using namespace cie;
   if (tokens <= 0) return 0;
   if (rot_dims % 2 || rot_dims > rot) CIE_FAIL("latent_prepare: %d rotated dims of %d", rot_dims, rot);
@@ -435,7 +437,7 @@ extern "C" int cie_latent_prepare(const float* down, int stride, void* q_out, co
     CIE_LAUNCH("latent_prepare", latent_prepare_kernel<T>, dim3(tokens), dim3(128), 0, (cudaStream_t)stream, down,
                stride, (T*)q_out, q_gain, kv_gain, positions, request_of_token, table, table_width, num_pages,
                (T*)c_pool, (T*)r_pool, inv_freq, magnitude, interleaved, rot_dims, q_rank, rank, rot, page_size,
-               eps, has_kv, write_cache, err);
+               eps, has_kv, write_cache, active, err);
   })
   return 0;
 }

@@ -4,7 +4,9 @@
 //              stored), a score function over all experts (softmax), the `top` largest of score +
 //              correction, and as mixing weights the scores of the chosen experts (optionally renormalised
 //              to sum 1); or (`chosen_softmax`) the `top` largest LOGITS and as weights the softmax over
-//              those logits alone
+//              those logits alone; or (`sigmoid`) the scores are sigmoids of the logits.  The experts may form equal
+//              groups of neighbours: a group's score is the sum of its two largest choice scores and only experts
+//              of the best groups can be chosen
 //   plan       counts per expert -> offsets; every (token, choice) pair gets a place in its expert's
 //              run of rows; runs are cut into tiles of 128 rows for the grouped products
 //   gate_up    rows gathered by place, times the expert's stacked gate and up matrices, SiLU(gate)*up
@@ -37,7 +39,7 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router,
                  const float* __restrict__ correction, int* __restrict__ ids,
                  float* __restrict__ weights, int* __restrict__ counts, int tokens,
                  int hidden, int experts, int top, int renormalize, const float* __restrict__ logit_bias,
-                 int chosen_softmax) {
+                 int chosen_softmax, int sigmoid, int groups, int keep_groups, float norm_floor) {
   extern __shared__ __align__(16) float score_s[];      // [2 * experts]: scores, then choice scores; then the row
   pdl_wait();
   pdl_trigger();
@@ -109,18 +111,44 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router,
     if (lane < top) weights[(size_t)t * top + lane] = mine / total;
     return;
   }
-  float m = -FLT_MAX;
-  for (int e = lane; e < experts; e += 32) m = fmaxf(m, score[e]);
-  m = warp_max(m);
-  float sum = 0.f;
-  for (int e = lane; e < experts; e += 32) sum += expf(score[e] - m);
-  sum = warp_sum(sum);
+  float m = 0.f, sum = 1.f;
+  if (!sigmoid) {
+    m = -FLT_MAX;
+    for (int e = lane; e < experts; e += 32) m = fmaxf(m, score[e]);
+    m = warp_max(m);
+    sum = 0.f;
+    for (int e = lane; e < experts; e += 32) sum += expf(score[e] - m);
+    sum = warp_sum(sum);
+  }
   for (int e = lane; e < experts; e += 32) {
-    const float s = expf(score[e] - m) / sum;
+    const float s = sigmoid ? 1.f / (1.f + expf(-score[e])) : expf(score[e] - m) / sum;
     score[e] = s;
     choice[e] = s + (correction ? correction[e] : 0.f);
   }
   __syncwarp();
+  if (keep_groups < groups) {
+    // a lane per group (in turns): the sum of the group's two largest choice scores
+    const int size = experts / groups;
+    float* strength = row_s;                    // the token's row is no longer needed
+    for (int g = lane; g < groups; g += 32) {
+      float first = -FLT_MAX, second = -FLT_MAX;
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float c = choice[e];
+        if (c > first) { second = first; first = c; }
+        else if (c > second) second = c;
+      }
+      strength[g] = size > 1 ? first + second : first;
+    }
+    __syncwarp();
+    // a group stays if fewer than keep_groups others are better (lowest index on ties)
+    for (int g = lane; g < groups; g += 32) {
+      int better = 0;
+      for (int o = 0; o < groups; ++o) better += strength[o] > strength[g] || (strength[o] == strength[g] && o < g);
+      if (better >= keep_groups)
+        for (int e = g * size; e < (g + 1) * size; ++e) choice[e] = -FLT_MAX;
+    }
+    __syncwarp();
+  }
   float chosen_sum = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -FLT_MAX;
@@ -142,7 +170,7 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router,
     chosen_sum += score[best_e];
     __syncwarp();
   }
-  if (renormalize && lane < top) weights[(size_t)t * top + lane] /= chosen_sum;
+  if (renormalize && lane < top) weights[(size_t)t * top + lane] /= chosen_sum + norm_floor;
 }
 
 // ---------------------------------------------------------------- plan
@@ -451,27 +479,34 @@ extern "C" int cie_moe_row_tile() { return kRowTile; }
 extern "C" int cie_moe_route(const void* x, const float* router, const float* correction, int* ids,
                              float* weights, int* counts, int* offsets, int* cursors, int* place_to_pair,
                              int* tiles, int* tile_count, int tokens, int hidden, int experts, int top,
-                             int renormalize, const float* logit_bias, int chosen_softmax, int dtype, void* stream) {
+                             int renormalize, const float* logit_bias, int chosen_softmax, int sigmoid, int groups,
+                             int keep_groups, float norm_floor, int dtype, void* stream) {
+  // sigmoid: scores are sigmoids of the logits; groups, keep_groups: experts in equal groups of which the best few can
+  // be chosen from (1, 1: all); norm_floor is added to the sum that the weights are divided by.
   if (tokens <= 0) return 0;
+  if (groups < 1 || experts % groups || keep_groups < 1 || keep_groups > groups)
+    CIE_FAIL("moe_route: %d of %d groups of %d experts", keep_groups, groups, experts);
+  if (top > experts / groups * keep_groups) CIE_FAIL("moe_route: top %d of the %d experts of the kept groups", top, experts / groups * keep_groups);
   if (experts < 1 || experts > kMaxExperts) CIE_FAIL("moe_route: 1..%d experts, got %d", kMaxExperts, experts);
   if (top < 1 || top > experts || top > 32) CIE_FAIL("moe_route: top %d of %d experts (at most 32)", top, experts);
   cudaStream_t s = (cudaStream_t)stream;
   if (cudaMemsetAsync(counts, 0, sizeof(int) * experts, s) != cudaSuccess) CIE_FAIL("moe_route: memset failed");
   const int warps = kRouteWarps;
-  const size_t smem = (size_t)(((2 * experts + 3) & ~3) + hidden) * sizeof(float);
+  const size_t smem = (size_t)(((2 * experts + 3) & ~3) + (hidden > groups ? hidden : groups)) * sizeof(float);
   if (smem > 200 * 1024) CIE_FAIL("moe_route: a row of %d elements does not fit shared memory", hidden);
   const int blocks = tokens;
   if (dtype == kFloat32) {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       CIE_FAIL("moe_route: cannot reserve %zu bytes of shared memory", smem);
     CIE_LAUNCH("moe_route", moe_route_kernel<float>, dim3(blocks), dim3(warps * 32), smem, s, (const float*)x, router,
-               correction, ids, weights, counts, tokens, hidden, experts, top, renormalize, logit_bias, chosen_softmax);
+               correction, ids, weights, counts, tokens, hidden, experts, top, renormalize, logit_bias, chosen_softmax, sigmoid,
+               groups, keep_groups, norm_floor);
   } else if (dtype == kBFloat16) {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       CIE_FAIL("moe_route: cannot reserve %zu bytes of shared memory", smem);
     CIE_LAUNCH("moe_route", moe_route_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, s,
                (const __nv_bfloat16*)x, router, correction, ids, weights, counts, tokens, hidden, experts, top,
-               renormalize, logit_bias, chosen_softmax);
+               renormalize, logit_bias, chosen_softmax, sigmoid, groups, keep_groups, norm_floor);
   } else {
     CIE_FAIL("moe_route: unknown element type code %d", dtype);
   }

@@ -155,11 +155,11 @@ mlstm_scan_kernel(const float* __restrict__ proj, int proj_stride, int q_off, in
 }
 
 // ---------------------------------------------------------------- short convolution + SiLU
-// out[t][c] = silu(sum_j w[c][j] * x[t - (taps - 1 - j)][c]) over the channels c < channels of `proj` (its first
-// columns), where x before the first token of this step comes from the request's history
+// out[t][c] = silu(sum_j w[c][j] * x[t - (taps - 1 - j)][c] + bias[c]) over the channels c < channels of `proj` (its
+// first columns; bias may be null), where x before the first token of this step comes from the request's history
 // hist[(taps - 1)][channels] (oldest first) and is zero at the start of a request.  grid (tokens, channel blocks).
 __global__ void short_conv_kernel(const float* __restrict__ proj, int proj_stride, const float* __restrict__ w,
-                                  int taps, const float* __restrict__ state, long long state_stride,
+                                  const float* __restrict__ bias, int taps, const float* __restrict__ state, long long state_stride,
                                   float* __restrict__ out, int out_stride, const int* __restrict__ query_start,
                                   const int* __restrict__ request_of_token, const int* __restrict__ slots,
                                   int channels, int max_slots, int* err) {
@@ -181,6 +181,38 @@ __global__ void short_conv_kernel(const float* __restrict__ proj, int proj_strid
     const float x = src >= 0 ? proj[(size_t)(begin + src) * proj_stride + c] : hist[(size_t)(taps - 1 + src) * channels + c];
     acc = fmaf(w[(size_t)c * taps + j], x, acc);
   }
+  if (bias) acc += bias[c];
+  out[(size_t)t * out_stride + c] = acc / (1.f + expf(-acc));
+}
+
+// The same for a step of single tokens (row t is request t): a thread reads its channel's history, writes the result
+// and moves the history on.
+__global__ void short_conv_single_kernel(const float* __restrict__ proj, int proj_stride, const float* __restrict__ w,
+                                         const float* __restrict__ bias, int taps, float* __restrict__ state,
+                                         long long state_stride, float* __restrict__ out, int out_stride,
+                                         const int* __restrict__ slots, const int* __restrict__ request_active,
+                                         int channels, int max_slots, int* err) {
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= channels) return;
+  const int slot = slots[t];
+  if (slot < 0 || slot >= max_slots) {
+    atomicOr(err, kErrBadRequest);
+    return;
+  }
+  const bool keep = request_active[t] != 0;
+  float* hist = state + (size_t)slot * state_stride;
+  const float now = proj[(size_t)t * proj_stride + c];
+  float acc = 0.f;
+  for (int j = 0; j < taps - 1; ++j) {
+    const float x = hist[(size_t)j * channels + c];
+    acc = fmaf(w[(size_t)c * taps + j], x, acc);
+    if (keep && j > 0) hist[(size_t)(j - 1) * channels + c] = x;
+  }
+  if (keep && taps > 1) hist[(size_t)(taps - 2) * channels + c] = now;
+  acc = fmaf(w[(size_t)c * taps + taps - 1], now, acc);
+  if (bias) acc += bias[c];
   out[(size_t)t * out_stride + c] = acc / (1.f + expf(-acc));
 }
 
@@ -1405,16 +1437,24 @@ extern "C" int cie_gated_delta_stream(const float* conv, int conv_stride, int q_
   return 0;
 }
 
-// The convolution of a step and then the history it leaves; `state` points at the history of slot 0.
-extern "C" int cie_short_conv(const float* proj, int proj_stride, const float* w, int taps, float* state,
+// The convolution of a step and then the history it leaves; `state` points at the history of slot 0.  bias: float32
+// [channels] or nullptr.  singles: every request brings one token (row t is request t).
+extern "C" int cie_short_conv(const float* proj, int proj_stride, const float* w, const float* bias, int taps, float* state,
                               long long state_stride, float* out, int out_stride, const int* query_start,
                               const int* request_of_token, const int* slots, const int* request_active, int tokens,
-                              int requests, int channels, int max_slots, int* err, void* stream) {
+                              int requests, int channels, int max_slots, int singles, int* err, void* stream) {
   if (tokens <= 0 || channels <= 0) return 0;
+  if (singles && tokens != requests) CIE_FAIL("short_conv: %d tokens of %d requests are not single tokens", tokens, requests);
   if (taps < 1 || taps > kMaxTaps) CIE_FAIL("short_conv: %d taps (1..%d)", taps, kMaxTaps);
   const int threads = 256, blocks = (channels + threads - 1) / threads;
+  if (singles) {
+    CIE_LAUNCH("short_conv", short_conv_single_kernel, dim3(tokens, blocks), dim3(threads), 0, (cudaStream_t)stream, proj,
+               proj_stride, w, bias, taps, state, state_stride, out, out_stride, slots, request_active, channels, max_slots,
+               err);
+    return 0;
+  }
   CIE_LAUNCH("short_conv", short_conv_kernel, dim3(tokens, blocks), dim3(threads), 0, (cudaStream_t)stream, proj,
-             proj_stride, w, taps, (const float*)state, state_stride, out, out_stride, query_start, request_of_token,
+             proj_stride, w, bias, taps, (const float*)state, state_stride, out, out_stride, query_start, request_of_token,
              slots, channels, max_slots, err);
   if (taps > 1)
     CIE_LAUNCH("short_conv_keep", short_conv_keep_kernel, dim3(requests, blocks), dim3(threads), 0,

@@ -1,0 +1,425 @@
+// State-space recurrence with ONE decay per head and token (Mamba-2's state-space duality):
+//
+//     dt_t = softplus(r_t + bias_h)                          (r: the projection's rate column of head h)
+//     S_t  = exp(-exp(A_h) * dt_t) S_(t-1) + dt_t * B_t x_t^T      S: [state][vdim], float32, per request and head
+//     y_t  = S_t^T C_t + D_h x_t
+//
+// Heads come in equal groups of neighbours that share B and C.  x, B and C arrive as float32 rows (after their short
+// convolution), the rate as a column of the projection.  Everything is float32.
+//
+// Single tokens (and any batch): `ssd_scan_kernel` walks the tokens with the state in registers.
+//
+// Prompt portions run in chunks of kChunk tokens.  With b_t = sum of the log decays from the chunk's first token to
+// t (all exponents below are <= 0):
+//   1. per (chunk, head)         dt_t and b_t                                            -> gates [T][heads][2]
+//   2. per (chunk, group)        G_ij = C_i . B_j for j <= i (shared by the group's heads)
+//   3. per (chunk, head)         U = sum_j exp(b_last - b_j) dt_j B_j x_j^T
+//   4. per (request, head)       walks its chunks, S <- exp(b_last) S + U, leaving the state BEFORE the chunk in U's
+//                                place; the last S goes to the slot
+//   5. per (chunk, head)         y_i = exp(b_i) S_before^T C_i + sum_(j<=i) exp(b_i - b_j) dt_j G_ij x_j + D x_i
+// Products 2, 3 and 5 are 64 x 64 tiles, four by four numbers a thread.  A request's result depends on its own tokens
+// and state only, whatever the batch or the slot, and on the cut of its prompt only through the order of additions.
+#include "common.cuh"
+
+CIE_DEFINE_LAST_ERROR()
+
+namespace cie {
+
+constexpr int kWarps = 8;
+constexpr int kMaxState = 256;
+constexpr int kChunk = 64;
+constexpr int kTile = 64;
+constexpr int kLd = kTile + 4;       // padded tile row: 16-byte pieces, few bank conflicts
+
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+// Columns of a float32 row: x (heads x vdim), B and C (groups x state) of `rows`; the rate of `proj`.
+struct Inputs {
+  const float* rows;
+  int stride, x_off, b_off, c_off;
+  const float* proj;
+  int proj_stride, r_off;
+  const float* a_log;
+  const float* dt_bias;
+  const float* skip;       // D
+  int heads, groups, state, vdim;
+};
+
+// ---------------------------------------------------------------- token by token
+// grid (requests, heads, ceil(vdim / 32)); warp w owns the state rows w, w + 8, ..., lane = value column.
+template <int R>
+__global__ void __launch_bounds__(kWarps * 32)
+ssd_scan_kernel(Inputs in, float* __restrict__ out, int out_stride, float* __restrict__ state, long long state_stride,
+                const int* __restrict__ query_start, const int* __restrict__ slots,
+                const int* __restrict__ request_active, int max_slots, int* err) {
+  __shared__ float b_s[2][kWarps * R], c_s[2][kWarps * R];
+  __shared__ float part_s[2][kWarps][32];
+  pdl_wait();
+  pdl_trigger();
+  const int request = blockIdx.x, head = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int column = blockIdx.z * 32 + lane, n = in.state;
+  const bool live = column < in.vdim;
+  const int slot = slots[request];
+  if (slot < 0 || slot >= max_slots) {
+    if (threadIdx.x == 0) atomicOr(err, kErrBadRequest);
+    return;
+  }
+  const int begin = query_start[request], end = query_start[request + 1];
+  const int group = head / (in.heads / in.groups);
+  const float rate = -expf(in.a_log[head]), bias = in.dt_bias[head], skip = in.skip[head];
+  float* s_base = state + (size_t)slot * state_stride + (size_t)head * n * in.vdim;
+  float s[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int i = warp + kWarps * r;
+    s[r] = (i < n && live) ? s_base[(size_t)i * in.vdim + column] : 0.f;
+  }
+  for (int t = begin; t < end; ++t) {
+    const int buf = (t - begin) & 1;
+    const float* row = in.rows + (size_t)t * in.stride;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      b_s[buf][i] = row[in.b_off + group * n + i];
+      c_s[buf][i] = row[in.c_off + group * n + i];
+    }
+    const float x = live ? row[in.x_off + head * in.vdim + column] : 0.f;
+    const float dt = softplus_f(in.proj[(size_t)t * in.proj_stride + in.r_off + head] + bias);
+    const float keep = expf(rate * dt), gained = dt * x;
+    __syncthreads();
+    float o = 0.f;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int i = warp + kWarps * r;
+      if (i < n) {
+        s[r] = fmaf(keep, s[r], b_s[buf][i] * gained);
+        o = fmaf(s[r], c_s[buf][i], o);
+      }
+    }
+    part_s[buf][warp][lane] = o;
+    __syncthreads();
+    if (warp == 0 && live) {
+      float total = 0.f;
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) total += part_s[buf][w][lane];
+      out[(size_t)t * out_stride + head * in.vdim + column] = fmaf(skip, x, total);
+    }
+    // the buffers of token t are written again only after the first barrier of token t + 2
+  }
+  if (request_active[request] && live) {
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int i = warp + kWarps * r;
+      if (i < n) s_base[(size_t)i * in.vdim + column] = s[r];
+    }
+  }
+}
+
+// ---------------------------------------------------------------- chunks
+// grid (chunks, ceil(heads / 128)): a thread a head walks the chunk's tokens.  gates: [T][heads] pairs (dt, b).
+__global__ void __launch_bounds__(128)
+ssd_gates_kernel(Inputs in, float2* __restrict__ gates, const int* __restrict__ chunk_row, const int* __restrict__ chunk_count) {
+  pdl_wait();
+  pdl_trigger();
+  const int head = blockIdx.y * 128 + threadIdx.x;
+  if (head >= in.heads) return;
+  const int row0 = chunk_row[blockIdx.x], n = chunk_count[blockIdx.x];
+  const float rate = -expf(in.a_log[head]), bias = in.dt_bias[head];
+  const float* r = in.proj + (size_t)row0 * in.proj_stride + in.r_off + head;
+  float sum = 0.f;
+  for (int j0 = 0; j0 < n; j0 += 8) {        // eight rates are asked for together
+    float dt[8];
+#pragma unroll
+    for (int u = 0; u < 8; ++u) dt[u] = j0 + u < n ? r[(size_t)(j0 + u) * in.proj_stride] : 0.f;
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      if (j0 + u >= n) break;
+      const float d = softplus_f(dt[u] + bias);
+      sum = fmaf(rate, d, sum);
+      gates[(size_t)(row0 + j0 + u) * in.heads + head] = make_float2(d, sum);
+    }
+  }
+}
+
+// acc[a][b] += sum over `depth` rows of left[k][4 ty + a] * right[k][4 tx + b]
+__device__ __forceinline__ void tile_product(float (&acc)[4][4], const float* left, const float* right, int depth, int ty, int tx) {
+#pragma unroll 4
+  for (int k = 0; k < depth; ++k) {
+    const float4 l = *reinterpret_cast<const float4*>(left + k * kLd + 4 * ty);
+    const float4 r = *reinterpret_cast<const float4*>(right + k * kLd + 4 * tx);
+    const float lv[4] = {l.x, l.y, l.z, l.w}, rv[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int a = 0; a < 4; ++a)
+#pragma unroll
+      for (int b = 0; b < 4; ++b) acc[a][b] = fmaf(lv[a], rv[b], acc[a][b]);
+  }
+}
+
+// dst[j][c] = src[(row0 + j)][col + c] * factor(j) for j < 64, c < 64; zero outside n rows and `width` columns.
+template <typename F>
+__device__ __forceinline__ void stage_rows(float* dst, const float* src, int stride, int row0, int n, int col, int width, F factor) {
+  if (((reinterpret_cast<uintptr_t>(src + (size_t)row0 * stride + col) & 15) == 0) && stride % 4 == 0 && width % 4 == 0) {
+#pragma unroll
+    for (int e = threadIdx.x; e < kTile * (kTile / 4); e += 256) {
+      const int j = e / (kTile / 4), c = (e % (kTile / 4)) * 4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (j < n && c < width) v = *reinterpret_cast<const float4*>(src + (size_t)(row0 + j) * stride + col + c);
+      const float f = factor(j);
+      *reinterpret_cast<float4*>(dst + j * kLd + c) = make_float4(v.x * f, v.y * f, v.z * f, v.w * f);
+    }
+    return;
+  }
+  for (int e = threadIdx.x; e < kTile * kTile; e += 256) {
+    const int j = e / kTile, c = e % kTile;
+    dst[j * kLd + c] = (j < n && c < width) ? src[(size_t)(row0 + j) * stride + col + c] * factor(j) : 0.f;
+  }
+}
+
+// dst[c][j] = src[(row0 + j)][col + c]: the same tile with tokens along the fast axis.  A thread takes one token's
+// piece of four columns; neighbouring threads take neighbouring tokens, so that the stores do not collide.
+__device__ __forceinline__ void stage_columns(float* dst, const float* src, int stride, int row0, int n, int col, int width) {
+  const bool wide = ((reinterpret_cast<uintptr_t>(src + (size_t)row0 * stride + col) & 15) == 0) && stride % 4 == 0 && width % 4 == 0;
+  for (int e = threadIdx.x; e < kTile * (kTile / 4); e += 256) {
+    const int j = e % kTile, c = (e / kTile) * 4;
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (j < n) {
+      const float* s = src + (size_t)(row0 + j) * stride + col + c;
+      if (wide && c < width) {
+        const float4 q = *reinterpret_cast<const float4*>(s);
+        v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+      } else {
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          if (c + x < width) v[x] = s[x];
+      }
+    }
+#pragma unroll
+    for (int x = 0; x < 4; ++x) dst[(c + x) * kLd + j] = v[x];
+  }
+}
+
+// G of a (chunk, group): products[chunk][group][j][i] = C_i . B_j (row j, so that step 5 reads it as it uses it).
+__global__ void __launch_bounds__(256)
+ssd_chunk_products_kernel(Inputs in, float* __restrict__ products, const int* __restrict__ chunk_row, const int* __restrict__ chunk_count) {
+  __shared__ __align__(16) float b_s[kTile * kLd], c_s[kTile * kLd];     // [state][token]
+  pdl_wait();
+  pdl_trigger();
+  const int chunk = blockIdx.x, group = blockIdx.y;
+  const int row0 = chunk_row[chunk], n = chunk_count[chunk];
+  const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+  float acc[4][4] = {};
+  for (int s0 = 0; s0 < in.state; s0 += kTile) {
+    const int width = min(kTile, in.state - s0);
+    stage_columns(b_s, in.rows, in.stride, row0, n, in.b_off + group * in.state + s0, width);
+    stage_columns(c_s, in.rows, in.stride, row0, n, in.c_off + group * in.state + s0, width);
+    __syncthreads();
+    tile_product(acc, b_s, c_s, width, ty, tx);
+    __syncthreads();
+  }
+  float* dst = products + ((size_t)chunk * in.groups + group) * kChunk * kChunk;
+#pragma unroll
+  for (int a = 0; a < 4; ++a)
+    *reinterpret_cast<float4*>(dst + (4 * ty + a) * kChunk + 4 * tx) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+}
+
+// U of a (chunk, head), tile by tile of [state][vdim].  grid (chunks, heads, state tiles * value tiles).
+__global__ void __launch_bounds__(256)
+ssd_chunk_sums_kernel(Inputs in, const float2* __restrict__ gates, float* __restrict__ sums,
+                      const int* __restrict__ chunk_row, const int* __restrict__ chunk_count) {
+  __shared__ __align__(16) float b_s[kTile * kLd], x_s[kTile * kLd];     // [token][state], [token][value]
+  __shared__ float w_s[kChunk];
+  pdl_wait();
+  pdl_trigger();
+  const int chunk = blockIdx.x, head = blockIdx.y;
+  const int value_tiles = (in.vdim + kTile - 1) / kTile;
+  const int s0 = blockIdx.z / value_tiles * kTile, v0 = blockIdx.z % value_tiles * kTile;
+  const int row0 = chunk_row[chunk], n = chunk_count[chunk];
+  const int group = head / (in.heads / in.groups);
+  if (threadIdx.x < kChunk) {
+    float w = 0.f;
+    if (threadIdx.x < n) {
+      const float2 g = gates[(size_t)(row0 + threadIdx.x) * in.heads + head];
+      w = expf(gates[(size_t)(row0 + n - 1) * in.heads + head].y - g.y) * g.x;
+    }
+    w_s[threadIdx.x] = w;
+  }
+  __syncthreads();
+  stage_rows(b_s, in.rows, in.stride, row0, n, in.b_off + group * in.state + s0, min(kTile, in.state - s0), [&](int j) { return w_s[j]; });
+  stage_rows(x_s, in.rows, in.stride, row0, n, in.x_off + head * in.vdim + v0, min(kTile, in.vdim - v0), [](int) { return 1.f; });
+  __syncthreads();
+  const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+  float acc[4][4] = {};
+  tile_product(acc, b_s, x_s, n, ty, tx);
+  float* dst = sums + ((size_t)chunk * in.heads + head) * in.state * in.vdim;
+#pragma unroll
+  for (int a = 0; a < 4; ++a) {
+    const int i = s0 + 4 * ty + a, c = v0 + 4 * tx;
+    if (i >= in.state) continue;
+    if (in.vdim % 4 == 0) {
+      if (c < in.vdim) *reinterpret_cast<float4*>(dst + (size_t)i * in.vdim + c) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+    } else {
+#pragma unroll
+      for (int b = 0; b < 4; ++b)
+        if (c + b < in.vdim) dst[(size_t)i * in.vdim + c + b] = acc[a][b];
+    }
+  }
+}
+
+// grid (requests, heads, blocks over state * vdim)
+__global__ void __launch_bounds__(256)
+ssd_chunk_walk_kernel(float* __restrict__ sums, float* __restrict__ state, long long state_stride,
+                      const float2* __restrict__ gates, const int* __restrict__ request_chunk_start,
+                      const int* __restrict__ chunk_row, const int* __restrict__ chunk_count, const int* __restrict__ slots,
+                      const int* __restrict__ request_active, int heads, int cells, int max_slots, int* err) {
+  pdl_wait();
+  pdl_trigger();
+  const int request = blockIdx.x, head = blockIdx.y;
+  const int e = blockIdx.z * blockDim.x + threadIdx.x;
+  if (e >= cells) return;
+  const int slot = slots[request];
+  if (slot < 0 || slot >= max_slots) {
+    if (e == 0) atomicOr(err, kErrBadRequest);
+    return;
+  }
+  float* cell = state + (size_t)slot * state_stride + (size_t)head * cells + e;
+  float s = *cell;
+  const size_t stride = (size_t)heads * cells;
+  const int last = request_chunk_start[request + 1];
+  constexpr int kBatch = 8;          // the sums of eight chunks are asked for together, before the first store
+  for (int chunk = request_chunk_start[request]; chunk < last; chunk += kBatch) {
+    float* u = sums + ((size_t)chunk * heads + head) * cells + e;
+    float gained[kBatch], power[kBatch];
+#pragma unroll
+    for (int b = 0; b < kBatch; ++b) {
+      const bool in = chunk + b < last;
+      gained[b] = in ? u[b * stride] : 0.f;
+      power[b] = in ? gates[(size_t)(chunk_row[chunk + b] + chunk_count[chunk + b] - 1) * heads + head].y : 0.f;
+    }
+#pragma unroll
+    for (int b = 0; b < kBatch; ++b) {
+      if (chunk + b < last) {
+        u[b * stride] = s;
+        s = fmaf(expf(power[b]), s, gained[b]);
+      }
+    }
+  }
+  if (request_active[request]) *cell = s;
+}
+
+// grid (chunks, heads, value tiles)
+__global__ void __launch_bounds__(256)
+ssd_chunk_output_kernel(Inputs in, const float2* __restrict__ gates, const float* __restrict__ products,
+                        const float* __restrict__ before_all, float* __restrict__ out, int out_stride,
+                        const int* __restrict__ chunk_row, const int* __restrict__ chunk_count) {
+  __shared__ __align__(16) float l_s[kTile * kLd], r_s[kTile * kLd];
+  __shared__ float dt_s[kChunk], b_s[kChunk];
+  pdl_wait();
+  pdl_trigger();
+  const int chunk = blockIdx.x, head = blockIdx.y, v0 = blockIdx.z * kTile;
+  const int row0 = chunk_row[chunk], n = chunk_count[chunk];
+  const int group = head / (in.heads / in.groups), width = min(kTile, in.vdim - v0);
+  if (threadIdx.x < kChunk) {
+    const float2 g = threadIdx.x < n ? gates[(size_t)(row0 + threadIdx.x) * in.heads + head] : make_float2(0.f, 0.f);
+    dt_s[threadIdx.x] = g.x;
+    b_s[threadIdx.x] = g.y;
+  }
+  const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+  const float* before = before_all + ((size_t)chunk * in.heads + head) * in.state * in.vdim;
+  float acc[4][4] = {};
+  for (int s0 = 0; s0 < in.state; s0 += kTile) {
+    const int depth = min(kTile, in.state - s0);
+    stage_columns(l_s, in.rows, in.stride, row0, n, in.c_off + group * in.state + s0, depth);
+    stage_rows(r_s, before, in.vdim, s0, depth, v0, width, [](int) { return 1.f; });
+    __syncthreads();
+    tile_product(acc, l_s, r_s, depth, ty, tx);
+    __syncthreads();
+  }
+  // what the state before the chunk gives decays to each token
+#pragma unroll
+  for (int a = 0; a < 4; ++a) {
+    const float carried = expf(b_s[4 * ty + a]);
+#pragma unroll
+    for (int b = 0; b < 4; ++b) acc[a][b] *= carried;
+  }
+  const float* g = products + ((size_t)chunk * in.groups + group) * kChunk * kChunk;
+  for (int e = threadIdx.x; e < kChunk * kChunk; e += 256) {
+    const int j = e / kChunk, i = e % kChunk;
+    l_s[j * kLd + i] = (j <= i && i < n) ? g[e] * (expf(b_s[i] - b_s[j]) * dt_s[j]) : 0.f;
+  }
+  stage_rows(r_s, in.rows, in.stride, row0, n, in.x_off + head * in.vdim + v0, width, [](int) { return 1.f; });
+  __syncthreads();
+  tile_product(acc, l_s, r_s, min(n, (4 * ty + 7) & ~3), ty, tx);      // tokens up to this thread's last one
+  const float skip = in.skip[head];
+#pragma unroll
+  for (int a = 0; a < 4; ++a) {
+    const int i = 4 * ty + a;
+    if (i >= n) continue;
+    float* dst = out + (size_t)(row0 + i) * out_stride + head * in.vdim + v0;
+#pragma unroll
+    for (int b = 0; b < 4; ++b)
+      if (4 * tx + b < width) dst[4 * tx + b] = fmaf(skip, r_s[i * kLd + 4 * tx + b], acc[a][b]);
+  }
+}
+
+}  // namespace cie
+
+using namespace cie;
+
+extern "C" int cie_ssd_max_state() { return kMaxState; }
+extern "C" int cie_ssd_chunk_tokens() { return kChunk; }
+
+// rows: float32 rows with x (heads * vdim), B and C (groups * state each) at the given columns; proj: rows with the
+// rates (heads) at r_off.  state: float32, slot after slot `state_stride` floats apart, heads [state][vdim] each.
+extern "C" int cie_ssd_scan(const float* rows, int stride, int x_off, int b_off, int c_off, const float* proj,
+                            int proj_stride, int r_off, const float* a_log, const float* dt_bias, const float* skip,
+                            float* out, int out_stride, float* state, long long state_stride, const int* query_start,
+                            const int* slots, const int* request_active, int requests, int heads, int groups, int n,
+                            int vdim, int max_slots, int* err, void* stream) {
+  if (requests <= 0) return 0;
+  if (n < 1 || n > kMaxState) CIE_FAIL("ssd_scan: a state of %d rows is outside 1..%d", n, kMaxState);
+  if (groups < 1 || heads < 1 || heads % groups || vdim < 1) CIE_FAIL("ssd_scan: %d heads of %d in %d groups", heads, vdim, groups);
+  const Inputs in{rows, stride, x_off, b_off, c_off, proj, proj_stride, r_off, a_log, dt_bias, skip, heads, groups, n, vdim};
+  const dim3 grid(requests, heads, (vdim + 31) / 32);
+#define CIE_SSD_SCAN(R)                                                                                              \
+  CIE_LAUNCH("ssd_scan", ssd_scan_kernel<R>, grid, dim3(kWarps * 32), 0, (cudaStream_t)stream, in, out, out_stride,  \
+             state, state_stride, query_start, slots, request_active, max_slots, err)
+  if (n <= 32) CIE_SSD_SCAN(4);
+  else if (n <= 64) CIE_SSD_SCAN(8);
+  else if (n <= 128) CIE_SSD_SCAN(16);
+  else CIE_SSD_SCAN(32);
+#undef CIE_SSD_SCAN
+  return 0;
+}
+
+// Floats of scratch memory: gates, products, sums.
+extern "C" long long cie_ssd_chunk_floats(int tokens, int chunks, int heads, int groups, int n, int vdim) {
+  const long long gates = ((long long)2 * tokens * heads + 3) / 4 * 4;
+  return gates + (long long)chunks * groups * kChunk * kChunk + (long long)chunks * heads * n * vdim;
+}
+
+extern "C" int cie_ssd_chunked(const float* rows, int stride, int x_off, int b_off, int c_off, const float* proj,
+                               int proj_stride, int r_off, const float* a_log, const float* dt_bias, const float* skip,
+                               float* out, int out_stride, float* state, long long state_stride, float* scratch,
+                               const int* chunk_row, const int* chunk_count, const int* request_chunk_start,
+                               const int* slots, const int* request_active, int tokens, int chunks, int requests,
+                               int heads, int groups, int n, int vdim, int max_slots, int* err, void* stream) {
+  if (chunks <= 0 || requests <= 0) return 0;
+  if (n < 1 || vdim < 1) CIE_FAIL("ssd_chunked: a state of %d x %d", n, vdim);
+  if (groups < 1 || heads < 1 || heads > 65535 || heads % groups) CIE_FAIL("ssd_chunked: %d heads in %d groups", heads, groups);
+  const Inputs in{rows, stride, x_off, b_off, c_off, proj, proj_stride, r_off, a_log, dt_bias, skip, heads, groups, n, vdim};
+  cudaStream_t s = (cudaStream_t)stream;
+  float2* gates = reinterpret_cast<float2*>(scratch);
+  float* products = scratch + ((long long)2 * tokens * heads + 3) / 4 * 4;
+  float* sums = products + (size_t)chunks * groups * kChunk * kChunk;
+  const int state_tiles = (n + kTile - 1) / kTile, value_tiles = (vdim + kTile - 1) / kTile;
+  CIE_LAUNCH("ssd_gates", ssd_gates_kernel, dim3(chunks, (heads + 127) / 128), dim3(128), 0, s, in, gates, chunk_row, chunk_count);
+  CIE_LAUNCH("ssd_chunk_products", ssd_chunk_products_kernel, dim3(chunks, groups), dim3(256), 0, s, in, products, chunk_row,
+             chunk_count);
+  CIE_LAUNCH("ssd_chunk_sums", ssd_chunk_sums_kernel, dim3(chunks, heads, state_tiles * value_tiles), dim3(256), 0, s, in,
+             (const float2*)gates, sums, chunk_row, chunk_count);
+  CIE_LAUNCH("ssd_chunk_walk", ssd_chunk_walk_kernel, dim3(requests, heads, (n * vdim + 255) / 256), dim3(256), 0, s, sums,
+             state, state_stride, (const float2*)gates, request_chunk_start, chunk_row, chunk_count, slots, request_active,
+             heads, n * vdim, max_slots, err);
+  CIE_LAUNCH("ssd_chunk_output", ssd_chunk_output_kernel, dim3(chunks, heads, value_tiles), dim3(256), 0, s, in,
+             (const float2*)gates, (const float*)products, (const float*)sums, out, out_stride, chunk_row, chunk_count);
+  return 0;
+}

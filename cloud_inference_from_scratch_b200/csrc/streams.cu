@@ -123,12 +123,26 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(float* __restrict__ st
 //   qk_norm  1: q and k are each divided by the root mean square of their WHOLE projection (all heads
 //            together) and multiplied by a gain vector of that size; 2: every head by its own root mean
 //            square, times a gain vector of a head's size that all heads share
+//            3: every head by its own root mean square AFTER the rotation, without a gain
 //   v_norm   every value head is divided by its own root mean square (no gain)
 //   rotation (inv_freq != nullptr) after the norms the first rot_dims elements of every q and k head turn by
 //            position * inv_freq[i], pair (i, i + rot_dims / 2) or, interleaved, (2i, 2i + 1); cos and sin
 //            are multiplied by `magnitude`; angle and rotation float32
+//   extra    q_factor: query head h is multiplied by q_factor[h] at the end; heat_every > 0: and by
+//            1 + heat * ln(floor((position + 1) / heat_every) + 1); v_mix 1: the token's values also go to `v_first`
+//            (float32 rows of kv_heads * vdim); 2: v becomes (1 - m) v + m v_first with m = *v_share
 // q goes to q_out (row stride q_stride); k and v go to their page slots
-// ([page][kv_head][page_size][dim or vdim]).
+// ([page][kv_head][page_size][dim or vdim]).  A request that is not active (`active`, may be null) writes nothing to
+// the pages: it only pads a batch, and with per-request state its rows may differ from those of the row it repeats.
+struct QkvExtra {
+  const float* q_factor;
+  float heat;
+  int heat_every;
+  float* v_first;
+  int v_mix;
+  const float* v_share;
+  const int* active;
+};
 template <typename TI, typename T>
 __global__ void norm_kv_write_kernel(const TI* __restrict__ src, const float* __restrict__ bias,
                                      T* __restrict__ q_out, int q_stride,
@@ -140,7 +154,7 @@ __global__ void norm_kv_write_kernel(const TI* __restrict__ src, const float* __
                                      int q_heads, int kv_heads, int dim, int vdim, int page_size,
                                      int qk_norm, int v_norm, float eps, int write_cache, int src_stride,
                                      const float* __restrict__ inv_freq, int rot_dims, float magnitude,
-                                     int interleaved, int* err) {
+                                     int interleaved, const QkvExtra extra, int* err) {
   extern __shared__ float row_s[];
   __shared__ float scratch[33];
   pdl_wait();
@@ -196,10 +210,38 @@ __global__ void norm_kv_write_kernel(const TI* __restrict__ src, const float* __
     }
     __syncthreads();
   }
+  if (qk_norm == 3) {
+    const int w = threadIdx.x >> 5, l = threadIdx.x & 31, ws = blockDim.x >> 5;
+    for (int h = w; h < q_heads + kv_heads; h += ws) {
+      float* head = row_s + (size_t)h * dim;
+      float sq = 0.f;
+      for (int d = l; d < dim; d += 32) sq = fmaf(head[d], head[d], sq);
+      const float inv = rsqrtf(warp_sum(sq) / (float)dim + eps);
+      for (int d = l; d < dim; d += 32) head[d] *= inv;
+    }
+    __syncthreads();
+  }
   T* q_row = q_out + (size_t)t * q_stride;
-  for (int i = threadIdx.x; i < q_width; i += blockDim.x) q_row[i] = from_float<T>(row_s[i]);
+  const float warmth = extra.heat_every > 0 ? 1.f + extra.heat * logf((float)((pos + 1) / extra.heat_every) + 1.f) : 1.f;
+  for (int i = threadIdx.x; i < q_width; i += blockDim.x) {
+    float v = row_s[i];
+    if (extra.heat_every > 0) v *= warmth;
+    if (extra.q_factor) v *= extra.q_factor[i / dim];
+    q_row[i] = from_float<T>(v);
+  }
+  if (extra.v_mix) {
+    float* v_row = row_s + q_width + k_width;
+    float* first = extra.v_first + (size_t)t * v_width;
+    const float share = extra.v_mix == 2 ? *extra.v_share : 0.f;
+    for (int i = threadIdx.x; i < v_width; i += blockDim.x) {
+      if (extra.v_mix == 1) first[i] = v_row[i];
+      else v_row[i] = fmaf(share, first[i], (1.f - share) * v_row[i]);
+    }
+    __syncthreads();
+  }
   if (!write_cache) return;
   const int request = request_of_token[t];
+  if (extra.active && !extra.active[request]) return;
   const int index = pos / page_size;
   const int page = index < table_width ? table[(size_t)request * table_width + index] : -1;
   if (page < 0 || page >= num_pages) {
@@ -305,13 +347,17 @@ extern "C" int cie_norm_kv_write(const void* src, const float* bias, void* q_out
                                  int kv_heads, int dim, int vdim, int page_size, int qk_norm, int v_norm,
                                  float eps, int write_cache, int src_stride, int src_dtype,
                                  const float* inv_freq, int rot_dims, float magnitude, int interleaved,
-                                 int dtype, int* err, void* stream) {
+                                 const float* q_factor, float heat, int heat_every, float* v_first, int v_mix,
+                                 const float* v_share, const int* active, int dtype, int* err, void* stream) {
   // qk_norm: 0 none; 1 over the whole projection (gains of the projection's size); 2 per head (gains of a
-  // head's size, shared by the heads).  src_stride: elements from one source row to the next (0: the
+  // head's size, shared by the heads); 3 per head after the rotation, no gains.  src_stride: elements from one source row to the next (0: the
   // row holds q, k and v and nothing else).  src_dtype: float32 or the activation type `dtype`.
   if (tokens <= 0) return 0;
-  if (qk_norm && (!q_gain || !k_gain)) CIE_FAIL("norm_kv_write: the q/k norm needs its gains");
-  if (qk_norm < 0 || qk_norm > 2) CIE_FAIL("norm_kv_write: unknown q/k norm %d", qk_norm);
+  if ((qk_norm == 1 || qk_norm == 2) && (!q_gain || !k_gain)) CIE_FAIL("norm_kv_write: the q/k norm needs its gains");
+  if (v_mix < 0 || v_mix > 2 || (v_mix && !v_first) || (v_mix == 2 && !v_share))
+    CIE_FAIL("norm_kv_write: mixing the values needs the first layer's and a share");
+  const QkvExtra extra{q_factor, heat, heat_every, v_first, v_mix, v_share, active};
+  if (qk_norm < 0 || qk_norm > 3) CIE_FAIL("norm_kv_write: unknown q/k norm %d", qk_norm);
   if (inv_freq && (rot_dims < 2 || rot_dims % 2 || rot_dims > dim))
     CIE_FAIL("norm_kv_write: %d rotated elements of a head of %d", rot_dims, dim);
   if (src_dtype != kFloat32 && src_dtype != dtype) CIE_FAIL("norm_kv_write: the source is float32 or of the activation type");
@@ -325,7 +371,8 @@ extern "C" int cie_norm_kv_write(const void* src, const float* bias, void* q_out
     CIE_LAUNCH("norm_kv_write", (norm_kv_write_kernel<TI, T>), dim3(tokens), dim3(256), smem, (cudaStream_t)stream, \
                (const TI*)src, bias, (T*)q_out, q_stride, positions, request_of_token, table, table_width,       \
                num_pages, (T*)k_pool, (T*)v_pool, q_gain, k_gain, q_heads, kv_heads, dim, vdim, page_size,       \
-               qk_norm, v_norm, eps, write_cache, src_stride, inv_freq, rot_dims, magnitude, interleaved, err);  \
+               qk_norm, v_norm, eps, write_cache, src_stride, inv_freq, rot_dims, magnitude, interleaved, extra, \
+               err);                                                                                            \
   } while (0)
   DISPATCH_DTYPE(dtype, "norm_kv_write", {
     if (src_dtype == kFloat32) CIE_NORM_KV(float, T);

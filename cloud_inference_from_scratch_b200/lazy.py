@@ -97,6 +97,32 @@ class NormedInput:
         return tuple(self.accumulated.scaled.shape)
 
 
+class NormedUpdate:
+    """A result ``y`` [T, H] that joins the residual stream RMS-normalised: ``x <- x + gain * y / rms(y)``, the root mean
+    square over the whole row with ``eps`` inside.  The norm that reads the stream next applies it in its own kernel,
+    in float32."""
+
+    def __init__(self, y: Any, gain: Any, eps: float) -> None:
+        self.y, self.gain, self.eps = y, gain, float(eps)
+
+    @property
+    def shape(self) -> tuple[int, ...]:
+        return tuple(self.y.shape)
+
+
+class PendingNorm:
+    """A norm that has not run yet, with what it needs: the stream, the update that still has to join it, gain, eps and
+    the number of parts.  Whoever takes this instead of a tensor (``takes_pending_norm``) runs the norm as the first
+    step of its own kernel."""
+
+    def __init__(self, residual: Any, update: Any, gain: Any, eps: float, groups: int) -> None:
+        self.residual, self.update, self.gain, self.eps, self.groups = residual, update, gain, float(eps), int(groups)
+
+    @property
+    def shape(self) -> tuple[int, ...]:
+        return tuple(self.residual.shape)
+
+
 class StreamUpdate:
     """A sublayer's result ``y`` [T, H] that has not been written to the residual streams yet: every
     stream t becomes ``sum_s mix[s, t] * stream_s + out[t] * y``.  ``mix`` None is the identity and

@@ -13,8 +13,8 @@ embedding rows (``position_tensor``), for a sinusoid of the position instead (``
 for several copies of the residual stream side by side (``residual_streams``, [T, streams * H]; the
 blocks of such a model read and write the copies and the final norm reads their sum), for a stored
 vector that is added to the stream right before a run of a layer (``ScheduleEntry.entry_offset``), for the
-embedding rows to be added once more there (``ScheduleEntry.adds_embedding``), and for a constant on every
-sublayer's result (``residual_scale``).
+embedding rows to be added once more there (``ScheduleEntry.adds_embedding``), for a constant on every
+sublayer's result (``residual_scale``), and for a norm on the embedding rows (``embedding_norm``).
 """
 
 from __future__ import annotations
@@ -96,6 +96,11 @@ class DecoderModel:
                 )
             )
         self.final_norm: Norm = build_part("norm", spec.final_norm)
+        self.embedding_norm: Any = None
+        if spec.embedding_norm is not None:
+            self.embedding_norm = build_part("norm", spec.embedding_norm)
+            if not hasattr(self.embedding_norm, "normalise_stream"):
+                raise ValueError(f"norm {spec.embedding_norm.kind!r} cannot normalise the embedding rows in place")
         # a projection may add itself into the residual stream only if whoever normalises next
         # understands that the sum is already there
         norms = [self.final_norm] + [part for layer in self.layers for slot, part in layer.parts.items()
@@ -132,6 +137,12 @@ class DecoderModel:
             for prefix, part in layer.named_parts():
                 for name, tensor in part.tensor_specs().items():
                     table[prefix + name] = tensor
+                for name, tensor in part.shared_tensor_specs().items():
+                    if table.setdefault(name, tensor) != tensor:
+                        raise ValueError(f"tensor {name!r} is shared by parts that disagree about it")
+        if self.embedding_norm is not None:
+            for name, tensor in self.embedding_norm.tensor_specs().items():
+                table[spec.embedding_norm_prefix + name] = tensor
         for name, tensor in self.final_norm.tensor_specs().items():
             table[spec.final_norm_prefix + name] = tensor
         return table
@@ -177,9 +188,20 @@ class DecoderModel:
             wave = torch.pow(torch.tensor(float(spec.position_wave_base), dtype=torch.float64),
                              -2.0 * pairs / spec.hidden_size)
             self.wave = wave.to(device=runtime.device, dtype=torch.float32).contiguous()
+        shared: dict[str, Any] = {}
         for layer in self.layers:
             for prefix, part in layer.named_parts():
                 part.bind({name: tensors(prefix + name) for name in part.tensor_specs()}, runtime)
+                wanted = part.shared_tensor_specs()
+                for name in wanted:
+                    if name not in shared:
+                        shared[name] = tensors(name)
+                if wanted:
+                    part.bind_shared({name: shared[name] for name in wanted})
+        if self.embedding_norm is not None:
+            self.embedding_norm.bind(
+                {name: tensors(spec.embedding_norm_prefix + name) for name in self.embedding_norm.tensor_specs()},
+                runtime)
         self.final_norm.bind(
             {name: tensors(spec.final_norm_prefix + name) for name in self.final_norm.tensor_specs()},
             runtime,
@@ -203,10 +225,13 @@ class DecoderModel:
                              positions=ctx.positions, position_table=self.position_table, streams=streams)
         else:
             rt.ops.embedding(ctx.token_ids, self.embedding, residual, spec.embedding_scale)
+        if self.embedding_norm is not None:
+            self.embedding_norm.normalise_stream(residual)
         embedded = None
         if any(entry.adds_embedding for entry in spec.schedule):
             # the stream as it is before the first layer, kept for the runs that add it again
-            if self.wave is not None or streams > 1 or self.position_table is not None:
+            if (self.wave is not None or streams > 1 or self.position_table is not None
+                    or self.embedding_norm is not None):
                 raise ValueError("adding the embedding rows again is built for a plain embedding")
             embedded = rt.workspace.get("embedded", ctx.num_tokens, spec.hidden_size, torch.float32)
             rt.ops.embedding(ctx.token_ids, self.embedding, embedded, spec.embedding_scale)

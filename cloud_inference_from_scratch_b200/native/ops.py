@@ -15,7 +15,7 @@ import os
 from ctypes import c_float, c_int, c_void_p
 from typing import Any
 
-from ..lazy import Accumulated, GateUpWeight, NormedInput, Partials, ResidualSink, StreamUpdate  # noqa: F401  (re-exported)
+from ..lazy import Accumulated, GateUpWeight, NormedInput, NormedUpdate, Partials, ResidualSink, StreamUpdate  # noqa: F401  (re-exported)
 from .build import load_library
 
 F32, BF16 = 0, 1
@@ -109,7 +109,7 @@ class Ops:
         ag = _Lib(load_library("attention_generic.cu"))
         self._attention_generic_sink = ag.function(
             "cie_attention_generic_sink",
-            [v, i, v, i, v, v, v, v, v, i, i, i, i, i, i, i, i, f, i, v, v, i, v, v, i, v, i, v, v],
+            [v, i, v, i, v, v, v, v, v, i, i, i, i, i, i, i, i, f, i, v, v, i, v, v, i, v, v, f, v, i, i, v, v],
         )
         self._group_share_floats = int(ag.handle.cie_attention_group_share_floats())
         self._group_tickets = None
@@ -121,6 +121,8 @@ class Ops:
         self._gla_lib = None
         self._recurrent_lib = None
         self._moe_lib = None
+        self._grouped_lib = None
+        self._ssd_lib = None
         self._sample = None   # sampling.cu is built when something is first sampled
         self._tensor_gemm = None
         self._fold_gemm_held = None
@@ -208,28 +210,30 @@ class Ops:
 
     def attention_penalised(self, q: Any, out: Any, ctx: Any, kv: Any, q_heads: int, kv_heads: int,
                             head_dim: int, value_dim: int, scale: float, window: int, distance: Any,
-                            keep_first: int = 0, sinks: Any = None) -> None:
-        """Attention with the options of ``attention_generic`` (a value size of its own, a distance
-        penalty, kept first keys), softmax weights float32 throughout.  bfloat16 prompt portions whose value heads have
-        the size of the key heads run on the tensor cores (mma.sync; the weights enter the value
-        product as two bfloat16 terms); single tokens, the 32-bit path and every other shape run on
-        the kernel that takes one warp per (token, head)."""
-        fast = (self._tensor_attention.get(head_dim)
-                if value_dim == head_dim and self.code == BF16 else None)
+                            keep_first: int = 0, sinks: Any = None, softcap: float = 0.0, slopes: Any = None,
+                            gates: Any = None) -> None:
+        """Attention with the options of ``attention_generic`` (a value size of its own, distance
+        penalties, a soft cap, kept first keys, sinks, a gate per head), softmax weights float32 throughout.  bfloat16
+        prompt portions whose key and value heads are multiples of 16 run on the tensor cores (mma.sync; the
+        weights enter the value product as two bfloat16 terms); single tokens, the 32-bit path and every other
+        shape run on the kernel whose heads of a group share the keys, or on one warp per (token, head)."""
+        fast = (self._tensor_attention.get(max(head_dim, value_dim))
+                if head_dim % 16 == 0 and value_dim % 16 == 0 and self.code == BF16 else None)
+        options = dict(keep_first=keep_first, sinks=sinks, softcap=softcap, slopes=slopes)
         singles = ctx.num_single
         if (fast is None or singles == ctx.num_requests or q.shape[1] % 8 or out.shape[1] % 8
                 or os.environ.get("CIE_PENALISED_TC", "1") == "0"):
             self.attention_generic(q, out, ctx, kv, q_heads, kv_heads, head_dim, scale, window,
                                    value_dim=value_dim, distance=distance,
-                                   few_tokens=singles == ctx.num_requests, keep_first=keep_first, sinks=sinks)
+                                   few_tokens=singles == ctx.num_requests, gates=gates, **options)
             return
         if singles:     # the leading rows of a mixed step are its single tokens
             self.attention_generic(q[:singles], out[:singles], ctx, kv, q_heads, kv_heads, head_dim, scale,
                                    window, value_dim=value_dim, distance=distance, few_tokens=True,
-                                   keep_first=keep_first, sinks=sinks)
+                                   gates=gates, **options)
         plan = ctx.extras.get(("attention", q_heads // kv_heads)) or None
-        fast.run_portions(q, out, ctx, kv, q_heads, kv_heads, scale, window, plan, distance, True,
-                          keep_first=keep_first, sinks=sinks)
+        fast.run_portions(q, out, ctx, kv, q_heads, kv_heads, scale, window, plan, distance, True, gates=gates,
+                          key_dim=head_dim, value_dim=value_dim, **options)
 
     def require_attention(self, head_dim: int) -> None:
         """Builds, at model set-up, the attention kernels a head size needs."""
@@ -412,7 +416,7 @@ class Ops:
                 "cie_mlstm_scan", [v, i, i, i, i, i, i, v, v, f, f, v, i, v, ll, v, v, v, i, i, i, i, i, v, v])
             self._gated_delta_scan = lib.function(
                 "cie_gated_delta_scan", [v, i, i, i, i, v, i, i, i, v, v, f, v, i, v, ll, v, v, v, i, i, i, i, i, i, v, v])
-            self._short_conv = lib.function("cie_short_conv", [v, i, v, i, v, ll, v, i, v, v, v, v, i, i, i, i, v, v])
+            self._short_conv = lib.function("cie_short_conv", [v, i, v, v, i, v, ll, v, i, v, v, v, v, i, i, i, i, i, v, v])
             self._head_norm_gate = lib.function("cie_head_norm_gate", [v, i, v, v, i, v, i, i, v, i, i, i, i, f, i, v])
             self._mlstm_stream = lib.function(
                 "cie_mlstm_stream", [v, i, i, i, i, i, i, v, v, f, f, v, v, i, v, v, ll, v, v, v, i, i, i, i, i, i, v, v])
@@ -517,18 +521,19 @@ class Ops:
                          ctx.num_requests, heads, dim, vdim, state.shape[0], _ptr(self.error_word), self.stream)
         return None
 
-    def short_conv(self, proj: Any, weight: Any, history: Any, out: Any, ctx: Any) -> None:
-        """out[t, c] = silu(sum_j weight[c, j] * x[t - (taps - 1 - j), c]) for the first ``weight.shape[0]``
-        columns of float32 ``proj``; inputs before this step come from ``history`` (a view [slots, (taps - 1) *
+    def short_conv(self, proj: Any, weight: Any, history: Any, out: Any, ctx: Any, bias: Any = None) -> None:
+        """out[t, c] = silu(sum_j weight[c, j] * x[t - (taps - 1 - j), c] + bias[c]) for the first ``weight.shape[0]``
+        columns of float32 ``proj`` (may be a view of columns); ``bias`` float32 or None; inputs before this step come from ``history`` (a view [slots, (taps - 1) *
         channels] of the requests' state, oldest first), which then takes this step's last inputs."""
         self._flush()
         self._load_recurrent()
         channels, taps = weight.shape
-        self.launches += 2 if taps > 1 else 1
-        self._short_conv(_ptr(proj), proj.stride(0), _ptr(weight), taps, _ptr(history), history.stride(0), _ptr(out),
-                         out.stride(0), _ptr(ctx.query_start), _ptr(ctx.request_of_token), _ptr(ctx.slots),
+        singles = proj.shape[0] == ctx.num_requests and ctx.num_single == ctx.num_requests
+        self.launches += 2 if taps > 1 and not singles else 1
+        self._short_conv(_ptr(proj), proj.stride(0), _ptr(weight), _ptr(bias), taps, _ptr(history), history.stride(0),
+                         _ptr(out), out.stride(0), _ptr(ctx.query_start), _ptr(ctx.request_of_token), _ptr(ctx.slots),
                          _ptr(ctx.request_active), proj.shape[0], ctx.num_requests, channels, history.shape[0],
-                         _ptr(self.error_word), self.stream)
+                         1 if singles else 0, _ptr(self.error_word), self.stream)
 
     def gated_delta_scan(self, conv: Any, offsets: tuple[int, int, int], proj: Any, gate_offsets: tuple[int, int],
                          a_log: Any, dt_bias: Any, q_scale: float, out: Any, state: Any, ctx: Any, heads: int,
@@ -596,6 +601,157 @@ class Ops:
                              _ptr(out), out.stride(0), out.shape[0], heads, size, float(eps), self._code_of(out),
                              self.stream)
 
+    # ------------------------------------------------------------------ norms in parts, and what sits beside them
+    def _load_grouped(self) -> None:
+        if self._grouped_lib is None:
+            v, i, f, ll = c_void_p, c_int, c_float, ctypes.c_longlong
+            lib = _Lib(load_library("grouped_norm.cu"))
+            self._group_norm = lib.function("cie_group_norm", [v, v, i, ll, v, f, v, v, v, i, i, i, f, i, i, v])
+            self._group_norm_conv = lib.function(
+                "cie_group_norm_conv",
+                [v, v, i, ll, v, f, v, v, v, v, i, v, ll, v, v, v, v, i, i, i, i, i, f, i, i, v, v])
+            self._gated_group_norm = lib.function("cie_gated_group_norm", [v, i, v, i, v, v, i, i, i, i, f, i, v])
+            self._side_gate = lib.function("cie_side_gate", [v, v, v, i, i, i, v, i, i, i, v, v])
+            self.norm_conv_max_taps = int(lib.handle.cie_norm_conv_max_taps())
+            self._grouped_lib = lib
+
+    def require_grouped(self) -> int:
+        """Builds, at model set-up, the kernels of norms in parts; returns the longest convolution they take."""
+        self._load_grouped()
+        return self.norm_conv_max_taps
+
+    def _pending_terms(self, update: Any) -> tuple[Any, int, int, Any, float]:
+        """A pending update as float32 terms: (tensor or None, terms, stride, gain or None, eps)."""
+        gain, eps = None, 0.0
+        if isinstance(update, NormedUpdate):
+            gain, eps, update = update.gain, update.eps, update.y
+        if isinstance(update, Accumulated):
+            raise KernelError("group_norm: an update that is already in the stream")
+        if isinstance(update, Partials) and (update.splits == 0 or update.bias is not None):
+            update = self.resolve(update, self.torch.empty(update.shape, dtype=self.torch.float32, device=self.device))
+        if update is None:
+            return None, 0, 0, None, 0.0
+        if isinstance(update, Partials):
+            return update.data, update.splits, update.stride, gain, eps
+        return (update if update.dtype == self.torch.float32 else update.float()), 1, 0, gain, eps
+
+    def group_norm(self, residual: Any, update: Any, gain: Any, eps: float, groups: int, out: Any, rows: Any = None) -> None:
+        """The pending update joins the float32 stream, and ``out`` is the norm of its rows in ``groups`` equal
+        consecutive parts, each divided by its own root mean square, times ``gain``; ``gain`` None: the rows
+        themselves, rounded.  ``update``: None, a tensor, ``Partials`` or a ``NormedUpdate``.  With ``rows`` only those
+        rows are read and the stream stays as it was.  ``out`` may be the stream itself."""
+        self._flush()
+        self._load_grouped()
+        count, hidden = out.shape
+        data, terms, stride, update_gain, update_eps = self._pending_terms(update)
+        self.launches += 1
+        self._group_norm(_ptr(residual), _ptr(data), terms, stride, _ptr(update_gain), float(update_eps), _ptr(gain),
+                         _ptr(out), _ptr(rows), count, hidden, groups, float(eps), 1 if gain is None else 0,
+                         self._code_of(out), self.stream)
+
+    def group_norm_conv(self, residual: Any, update: Any, gain: Any, eps: float, groups: int, weight: Any, history: Any,
+                        out: Any, ctx: Any) -> None:
+        """``group_norm`` and then ``out_t = h_t + sum_j weight[:, j] * h_(t - taps + 1 + j)`` over the normalised rows h of
+        every request (zeros before its first token; ``history``: float32 view [slots, (taps - 1) * H] of the requests'
+        state, oldest first, None for one tap).  Nothing is rounded between the norm and the convolution."""
+        self._flush()
+        self._load_grouped()
+        tokens, hidden = out.shape
+        taps = weight.shape[1]
+        data, terms, stride, update_gain, update_eps = self._pending_terms(update)
+        singles = tokens == ctx.num_requests and ctx.num_single == ctx.num_requests
+        inverses = None
+        if not singles:
+            inverses = self.scratch(f"norm_conv.inverses.{groups}", tokens * groups,
+                                    reserve=max(tokens, self.max_rows) * groups)
+        self.launches += 1 if singles else (3 if taps > 1 else 2)
+        self._group_norm_conv(_ptr(residual), _ptr(data), terms, stride, _ptr(update_gain), float(update_eps), _ptr(gain),
+                              _ptr(out), _ptr(inverses), _ptr(weight), taps, _ptr(history),
+                              history.stride(0) if history is not None else 0, _ptr(ctx.query_start),
+                              _ptr(ctx.request_of_token), _ptr(ctx.slots), _ptr(ctx.request_active), tokens,
+                              ctx.num_requests, history.shape[0] if history is not None else 1 << 30, hidden, groups,
+                              float(eps), 1 if singles else 0, self._code_of(out), _ptr(self.error_word), self.stream)
+
+    def gated_group_norm(self, y: Any, z: Any, gain: Any, eps: float, groups: int, out: Any) -> None:
+        """u = y * silu(z) (float32 rows, views of columns allowed), every one of ``groups`` equal parts of u divided by
+        its own root mean square, times ``gain``."""
+        self._flush()
+        self._load_grouped()
+        self.launches += 1
+        self._gated_group_norm(_ptr(y), y.stride(0), _ptr(z), z.stride(0), _ptr(gain), _ptr(out), out.stride(0), out.shape[0],
+                               out.shape[1], groups, float(eps), self._code_of(out), self.stream)
+
+    def side_gate(self, z: Any, token_ids: Any, table: Any, column: int, out: Any) -> None:
+        """out[t] = gelu_tanh(z[t]) * table[token_ids[t], column : column + out.shape[1]]; ``z`` contiguous float32,
+        ``table`` of ``out``'s dtype."""
+        self._flush()
+        self._load_grouped()
+        self.launches += 1
+        self._side_gate(_ptr(z), _ptr(token_ids), _ptr(table), table.shape[1], table.shape[0], int(column), _ptr(out),
+                        out.shape[0], out.shape[1], self._code_of(out), _ptr(self.error_word), self.stream)
+
+    # ------------------------------------------------------------------ state-space recurrence
+    def _load_ssd(self) -> None:
+        if self._ssd_lib is None:
+            v, i, ll = c_void_p, c_int, ctypes.c_longlong
+            lib = _Lib(load_library("ssd.cu"))
+            self._ssd_scan = lib.function(
+                "cie_ssd_scan", [v, i, i, i, i, v, i, i, v, v, v, v, i, v, ll, v, v, v, i, i, i, i, i, i, v, v])
+            self._ssd_chunked = lib.function(
+                "cie_ssd_chunked",
+                [v, i, i, i, i, v, i, i, v, v, v, v, i, v, ll, v, v, v, v, v, v, i, i, i, i, i, i, i, i, v, v])
+            lib.handle.cie_ssd_chunk_floats.restype = ctypes.c_longlong
+            self._ssd_chunk_floats = lib.handle.cie_ssd_chunk_floats
+            self.ssd_max_state = int(lib.handle.cie_ssd_max_state())
+            self.ssd_chunk_tokens = int(lib.handle.cie_ssd_chunk_tokens())
+            self._ssd_lib = lib
+
+    def require_ssd(self) -> int:
+        """Builds, at model set-up, the kernels of the state-space recurrence; returns the largest state size they take."""
+        self._load_ssd()
+        return self.ssd_max_state
+
+    def plan_ssd(self, host: Any) -> dict[str, Any]:
+        """Chunk work lists of the state-space recurrence for a step that holds prompt portions (one list serves every
+        such layer); a step of single tokens needs none."""
+        if host.num_single == host.num_requests:
+            return {}
+        self._load_ssd()
+        return self._plan_chunks(host, self.ssd_chunk_tokens)
+
+    def ssd(self, rows: Any, offsets: tuple[int, int, int], rates: Any, a_log: Any, dt_bias: Any, skip: Any, out: Any,
+            state: Any, ctx: Any, heads: int, groups: int, dim: int, vdim: int, plan: dict[str, Any] | None = None) -> None:
+        """The state-space recurrence over every request's new tokens from the state in its slot (``state``: float32,
+        at least heads * dim * vdim numbers a slot, a head's [dim, vdim] after the other):
+        ``S <- exp(-exp(a_log) dt) S + dt B x^T``, ``y = S^T C + skip x`` with ``dt = softplus(rate + dt_bias)``.
+        ``rows`` float32 [T, *] with x (heads * vdim), B and C (groups * dim) at the columns ``offsets``; ``rates``
+        float32, a view of [T, heads] columns; ``out`` float32 [T, heads * vdim].  With ``plan`` (``plan_ssd``, on the
+        device) and eight tokens a request or more on average the step runs in chunks, else token by token."""
+        self._flush()
+        self._load_ssd()
+        tokens = rows.shape[0]
+        head = (_ptr(rows), rows.stride(0), int(offsets[0]), int(offsets[1]), int(offsets[2]), _ptr(rates), rates.stride(0), 0,
+                _ptr(a_log), _ptr(dt_bias), _ptr(skip), _ptr(out), out.stride(0), _ptr(state), state.stride(0))
+        chunks = plan["chunk_row"].shape[0] if plan else 0
+        tag = f"ssd.chunks.{heads}x{groups}x{dim}x{vdim}"
+        floats = int(self._ssd_chunk_floats(tokens, chunks, heads, groups, dim, vdim))
+        held = self._partial_buffers.get(tag)
+        # under captured graphs the scratch memory keeps its place: a step of more chunks than it holds scans
+        fits = not self.scratch_frozen or held is None or held.numel() >= floats
+        if chunks and fits and tokens >= 8 * ctx.num_requests and os.environ.get("CIE_SSD_CHUNKS", "1") != "0":
+            # room for the chunks of the largest step the runtime knows of (and a partial chunk for many requests)
+            most = max(tokens, self.max_rows)
+            reserve = int(self._ssd_chunk_floats(most, -(-most // self.ssd_chunk_tokens) + 64, heads, groups, dim, vdim))
+            scratch = self.scratch(tag, floats, reserve=max(floats, reserve))
+            self.launches += 5
+            self._ssd_chunked(*head, _ptr(scratch), _ptr(plan["chunk_row"]), _ptr(plan["chunk_count"]),
+                              _ptr(plan["request_chunk_start"]), _ptr(ctx.slots), _ptr(ctx.request_active), tokens, chunks,
+                              ctx.num_requests, heads, groups, dim, vdim, state.shape[0], _ptr(self.error_word), self.stream)
+            return
+        self.launches += 1
+        self._ssd_scan(*head, _ptr(ctx.query_start), _ptr(ctx.slots), _ptr(ctx.request_active), ctx.num_requests, heads,
+                       groups, dim, vdim, state.shape[0], _ptr(self.error_word), self.stream)
+
     # ------------------------------------------------------------------ residual streams
     def _load_streams(self) -> None:
         if self._streams_lib is None:
@@ -605,7 +761,8 @@ class Ops:
             self._stream_norm = lib.function("cie_stream_norm", [v, i, v, i, v, v, v, v, i, v, v, i, i, f, i, v])
             self._norm_kv_write = lib.function(
                 "cie_norm_kv_write",
-                [v, v, v, i, v, v, v, i, i, v, v, v, v, i, i, i, i, i, i, i, i, f, i, i, i, v, i, f, i, i, v, v])
+                [v, v, v, i, v, v, v, i, i, v, v, v, v, i, i, i, i, i, i, i, i, f, i, i, i, v, i, f, i, v, f, i, v, i, v, v,
+                 i, v, v])
             self._streams_lib = lib
 
     def stream_norm(self, residual: Any, streams: int, update: Any, read: Any, gain: Any, eps: float,
@@ -636,7 +793,9 @@ class Ops:
 
     def norm_kv_write(self, qkv: Any, ctx: Any, kv: Any, q_heads: int, kv_heads: int, dim: int, vdim: int,
                       q_gain: Any, k_gain: Any, value_norm: bool, eps: float, q_buffer: Any,
-                      write_cache: bool = True, per_head: bool = False, rotation: Any = None) -> Any:
+                      write_cache: bool = True, per_head: bool = False, rotation: Any = None,
+                      unit_heads: bool = False, q_factor: Any = None, heat: tuple[float, int] | None = None,
+                      first_values: Any = None, value_share: Any = None) -> Any:
         """q and k of every token divided by the root mean square of their whole projection and
         multiplied by a gain vector (``q_gain`` None: left as they are), every value head divided by
         its own root mean square (``value_norm``); q goes to ``q_buffer``, k and v into the pages.
@@ -644,6 +803,11 @@ class Ops:
         are vectors of a head's size that all heads share.
         ``rotation`` (``inv_freq`` float32 [dims / 2], ``dims``, ``magnitude``, ``interleaved``): after the norms
         the first ``dims`` elements of every q and k head turn by the token's position.
+        ``unit_heads``: after the rotation every q and k head is divided by its own root mean square, without gains.
+        ``q_factor`` (float32 [q_heads]) multiplies the query heads; ``heat`` = (coef, every) multiplies q by
+        ``1 + coef * ln(floor((p + 1) / every) + 1)`` at position p.  ``first_values`` (float32 [T, kv_heads * vdim]):
+        takes this step's values if ``value_share`` is None, else v becomes ``(1 - m) v + m * first_values`` with
+        m the number in ``value_share``.  Requests that only pad the batch write nothing to the pages.
         ``qkv`` is a tensor [T, (Hq + Hkv) * dim + Hkv * vdim] of the compute dtype or of float32 (its rows may
         go on with other columns, which are left alone) or ``Partials`` with its bias pending."""
         self._flush()
@@ -659,13 +823,16 @@ class Ops:
         self._norm_kv_write(_ptr(qkv), _ptr(bias), _ptr(q_buffer), q_buffer.shape[1], _ptr(ctx.positions),
                             _ptr(ctx.request_of_token), _ptr(table), table.shape[1], kv.num_pages, _ptr(kv.k),
                             _ptr(kv.v), _ptr(q_gain), _ptr(k_gain), qkv.shape[0], q_heads, kv_heads, dim, vdim,
-                            kv.page_size, 0 if q_gain is None else (2 if per_head else 1), 1 if value_norm else 0,
+                            kv.page_size, 3 if unit_heads else (0 if q_gain is None else (2 if per_head else 1)),
+                            1 if value_norm else 0,
                             float(eps), 1 if write_cache else 0, qkv.stride(0), self._code_of(qkv),
                             _ptr(rotation.inv_freq) if rotation is not None else None,
                             int(rotation.dims) if rotation is not None else 0,
                             float(rotation.magnitude) if rotation is not None else 1.0,
                             int(rotation.interleaved) if rotation is not None else 0,
-                            self._code_of(q_buffer), _ptr(self.error_word), self.stream)
+                            _ptr(q_factor), float(heat[0]) if heat else 0.0, int(heat[1]) if heat else 0,
+                            _ptr(first_values), 0 if first_values is None else (1 if value_share is None else 2),
+                            _ptr(value_share), _ptr(getattr(ctx, "request_active", None)), self._code_of(q_buffer), _ptr(self.error_word), self.stream)
         return q_buffer
 
     # ------------------------------------------------------------------ linear attention with decay
@@ -814,7 +981,7 @@ class Ops:
             v, i, f = c_void_p, c_int, c_float
             lib = _Lib(load_library("latent.cu"))
             self._latent_prepare = lib.function(
-                "cie_latent_prepare", [v, i, v, v, v, v, v, v, i, i, v, v, v, f, i, i, i, i, i, i, i, f, i, i, i, v, v])
+                "cie_latent_prepare", [v, i, v, v, v, v, v, v, i, i, v, v, v, f, i, i, i, i, i, i, i, f, i, i, v, i, v, v])
             self._head_linear = lib.function("cie_head_linear", [v, i, i, v, v, i, i, v, i, i, i, i, i, i, i, v])
             self._latent_attention = lib.function(
                 "cie_latent_attention",
@@ -852,7 +1019,8 @@ class Ops:
                              _ptr(ctx.request_of_token), _ptr(table), table.shape[1], kv.num_pages, _ptr(kv.k),
                              _ptr(kv.v), _ptr(rotation.inv_freq), float(rotation.magnitude), int(rotation.interleaved),
                              int(rotation.dims), down.shape[0], q_rank, rank, rot, kv.page_size, float(eps),
-                             1 if has_kv else 0, 1 if write_cache else 0, self.code, _ptr(self.error_word), self.stream)
+                             1 if has_kv else 0, 1 if write_cache else 0, _ptr(getattr(ctx, "request_active", None)), self.code,
+                             _ptr(self.error_word), self.stream)
 
     def head_linear(self, x: Any, x_head: int, weight: Any, out: Any, out_head: int, heads: int, gate: Any = None) -> None:
         """A product per head: ``out[t, h, :N] = x[t, h, :K] @ weight[h]`` with ``weight`` [heads, K, N] in
@@ -1021,9 +1189,9 @@ class Ops:
     # ------------------------------------------------------------------ routed experts
     def _load_moe(self) -> None:
         if self._moe_lib is None:
-            v, i = c_void_p, c_int
+            v, i, f = c_void_p, c_int, c_float
             lib = _Lib(load_library("moe.cu"))
-            self._moe_route = lib.function("cie_moe_route", [v, v, v, v, v, v, v, v, v, v, v, i, i, i, i, i, v, i, i, v])
+            self._moe_route = lib.function("cie_moe_route", [v, v, v, v, v, v, v, v, v, v, v, i, i, i, i, i, v, i, i, i, i, f, i, v])
             self._moe_gate_up_simt = lib.function("cie_moe_gate_up_simt", [v, v, v, v, v, v, v, i, i, i, i, i, i, v])
             self._moe_down_simt = lib.function("cie_moe_down_simt", [v, v, v, v, v, v, i, i, i, i, i, i, v])
             self._moe_combine = lib.function("cie_moe_combine", [v, v, v, i, i, i, i, v])
@@ -1057,12 +1225,16 @@ class Ops:
 
     def routed_experts(self, x: Any, router: Any, correction: Any, w_gate: Any, w_up: Any, w_down: Any,
                        top: int, renormalize: bool, out: Any, workspace: Any, router_bias: Any = None,
-                       chosen_softmax: bool = False) -> Any:
+                       chosen_softmax: bool = False, sigmoid: bool = False, groups: tuple[int, int] = (1, 1),
+                       norm_floor: float = 0.0) -> Any:
         """out[t] = sum over the ``top`` chosen experts e of score_e * down_e(SiLU(gate_e x) * up_e x).
         ``router`` float32 [E, H]; ``w_gate``/``w_up`` [E, F, H], or ``w_up`` None and ``w_gate`` the
         interleaved [E, 2F, H] of ``interleave_gate_up``; ``w_down`` [E, H, F]; ``out`` float32 or the
         activation type.  ``router_bias`` (float32 [E]) is added to the router's logits; ``chosen_softmax``: the
-        experts with the largest logits are chosen and weighted by the softmax over their logits alone."""
+        experts with the largest logits are chosen and weighted by the softmax over their logits alone;
+        ``sigmoid``: scores are sigmoids of the logits; ``groups`` = (count, keep): experts form equal groups of
+        neighbours and only those of the ``keep`` groups whose two largest choice scores have the largest sums can
+        be chosen; ``norm_floor`` is added to the sum that ``renormalize`` divides by."""
         self._flush()
         self._load_moe()
         torch = self.torch
@@ -1086,7 +1258,7 @@ class Ops:
         self._moe_route(_ptr(x), _ptr(router), _ptr(correction), _ptr(ids), _ptr(weights), _ptr(counts),
                         _ptr(offsets), _ptr(cursors), _ptr(place_to_pair), _ptr(tiles), _ptr(tile_count), tokens,
                         hidden, experts, top, 1 if renormalize else 0, _ptr(router_bias), 1 if chosen_softmax else 0,
-                        code, self.stream)
+                        1 if sigmoid else 0, groups[0], groups[1], float(norm_floor), code, self.stream)
         aligned = (x.data_ptr() | w_gate.data_ptr() | w_down.data_ptr() | act.data_ptr()) % 16 == 0
         if w_up is None and not (code == BF16 and aligned):
             raise KernelError("routed_experts: interleaved gate/up weights are for aligned bfloat16 operands")
@@ -1463,11 +1635,15 @@ class Ops:
     def attention_generic(self, qkv: Any, out: Any, ctx: Any, kv: Any, q_heads: int,
                           kv_heads: int, head_dim: int, scale: float, window: int,
                           value_dim: int | None = None, distance: Any = None, few_tokens: bool = False,
-                          keep_first: int = 0, sinks: Any = None) -> None:
+                          keep_first: int = 0, sinks: Any = None, softcap: float = 0.0, slopes: Any = None,
+                          gates: Any = None) -> None:
         """``keep_first``: with a window, the request's first so many keys stay visible behind it.
         ``value_dim``: size of a value head when it is not ``head_dim``; ``distance``: (r1, r2),
         float32 [q_heads] each, of the penalty r1 * log(1 + r2 * (query position - key position)).
         ``sinks``: float32 [q_heads]; exp(sinks[h]) joins the softmax denominator of head h.
+        ``softcap`` > 0: the scaled score s becomes softcap * tanh(s / softcap); ``slopes`` (float32 [q_heads]): it is
+        then lowered by slopes[h] * distance; ``gates`` (float32, a view of [T, q_heads] columns): head h's output
+        is multiplied by sigmoid(gates[t, h]).
         ``few_tokens``: the rows are single tokens of a decode step; their keys are then cut into
         ranges with a CTA each where the device would otherwise stand mostly idle."""
         self._flush()
@@ -1493,7 +1669,8 @@ class Ops:
             _ptr(qkv), qkv.shape[1], _ptr(out), out.shape[1], _ptr(kv.k), _ptr(kv.v), _ptr(ctx.positions),
             _ptr(ctx.request_of_token), _ptr(table), table.shape[1], kv.num_pages, tokens, q_heads, kv_heads,
             head_dim, value_dim or head_dim, kv.page_size, scale, window, _ptr(r1), _ptr(r2), splits,
-            _ptr(shares), _ptr(tickets), int(keep_first), _ptr(sinks), self._code_of(qkv),
+            _ptr(shares), _ptr(tickets), int(keep_first), _ptr(sinks), _ptr(slopes), float(softcap), _ptr(gates),
+            gates.stride(0) if gates is not None else 0, self._code_of(qkv),
             _ptr(self.error_word), self.stream)
 
     def silu_mul(self, gate_up: Any, out: Any, block: int | None = None) -> None:

@@ -92,7 +92,7 @@ class TensorAttention:
         )
         self._prefill_ex = lib.function(
             "cie_attention_prefill_ex",
-            [v, i, v, i, v, v, v, i, i, v, v, i, v, v, v, i, i, i, i, f, i, v, v, i, i, v, v, v],
+            [v, i, v, i, v, v, v, i, i, v, v, i, v, v, v, i, i, i, i, f, i, v, v, i, i, v, i, i, f, v, v, i, v, v],
         )
         self._decode = lib.function(
             "cie_attention_decode",
@@ -330,12 +330,15 @@ class TensorAttention:
 
     def run_portions(self, qkv: Any, out: Any, ctx: Any, kv: Any, q_heads: int, kv_heads: int, scale: float,
                      window: int, plan: dict[str, Any] | None, distance: Any, split_weights: bool,
-                     keep_first: int = 0, sinks: Any = None) -> None:
+                     keep_first: int = 0, sinks: Any = None, softcap: float = 0.0, slopes: Any = None,
+                     gates: Any = None, key_dim: int | None = None, value_dim: int | None = None) -> None:
         """The prompt portions of a step (every request after the leading single tokens) on the
         mma.sync kernel, with the options the other kernels do not have: a distance penalty
         (``distance``: float32 vectors r1, r2 per query head), softmax weights that enter the value
-        product as two bfloat16 terms, a request's first ``keep_first`` keys visible behind the window, and a
-        sink term per query head in the softmax denominator (``sinks``: float32 [q_heads])."""
+        product as two bfloat16 terms, a request's first ``keep_first`` keys visible behind the window, a
+        sink term per query head in the softmax denominator (``sinks``: float32 [q_heads]), a soft cap on the scores,
+        a penalty ``slopes[h] * distance``, a sigmoid gate per head on the output, and key and value heads of their
+        own sizes (``key_dim``, ``value_dim``: multiples of 16 up to this build's head size)."""
         ops = self.ops
         torch = ops.torch
         table = ctx.block_tables[kv.group]
@@ -353,6 +356,9 @@ class TensorAttention:
                          ctx.query_start.data_ptr(), q_heads, kv_heads, kv.page_size, heads_per_tile(group),
                          scale, window, None if r1 is None else r1.data_ptr(), None if r2 is None else r2.data_ptr(),
                          1 if split_weights else 0, int(keep_first), None if sinks is None else sinks.data_ptr(),
+                         key_dim or self.head_dim, value_dim or self.head_dim, float(softcap),
+                         None if slopes is None else slopes.data_ptr(), None if gates is None else gates.data_ptr(),
+                         0 if gates is None else gates.stride(0),
                          ops.error_word.data_ptr(), ops.stream)
 
     def run(self, qkv: Any, out: Any, ctx: Any, kv: Any, q_heads: int, kv_heads: int,

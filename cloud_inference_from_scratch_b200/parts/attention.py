@@ -31,6 +31,16 @@ Options beyond the reference, each a constant of the part so that any descriptio
   ``r1_h * ln(1 + r2_h * (i - j))`` with two stored numbers per query head;
 * ``sink``: the softmax denominator of every query head holds one more term ``exp(sink_h)``, a stored number
   per head that has no key and no value and is not scaled;
+  (``sink="one"``: the term is ``exp(0)`` for every head and nothing is stored);
+* ``qk_norm="unit"``: every q and k head is divided by its own root mean square AFTER the rotation, without gains;
+* ``query_heat`` = (coef, every): q is multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)`` at position p;
+* ``head_factor``: the scores of every query head are multiplied by a stored number (before a cap);
+* ``softcap`` c > 0: the scaled score s becomes ``c * tanh(s / c)``;
+* ``distance_slopes``: the score is then lowered by ``2^(-8 (h + 1) / H) * (i - j)`` for query head h of H;
+* ``head_gate``: query head h's output is multiplied by ``sigmoid(W_g x)_h``, one number a head (the gate's weight is
+  stacked under q, k and v), before the output projection;
+* ``value_mix`` "keep": the layer's values are also kept for later layers of the same step; "blend": its values v become
+  ``(1 - m) v + m * kept`` with a stored number m before they are cached (both store ``m``; "keep" does not use it);
 * ``projection_float32``: q, k and v leave their product as float32 and are not rounded before the norms and
   the rotation;
 * ``position=None``: no rotation;
@@ -71,6 +81,12 @@ class Attention(Mixer):
         gate: bool = False,
         sink: bool = False,
         projection_float32: bool = False,
+        query_heat: tuple[float, int] | None = None,
+        head_factor: bool = False,
+        softcap: float = 0.0,
+        distance_slopes: bool = False,
+        head_gate: bool = False,
+        value_mix: str | None = None,
     ) -> None:
         if num_heads % num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
@@ -84,7 +100,21 @@ class Attention(Mixer):
         if keep_first < 0:
             raise ValueError("keep_first must not be negative")
         self.gate = bool(gate)
-        self.sink = bool(sink)
+        if sink not in (False, True, "one"):
+            raise ValueError(f"sink must be False, True or 'one', got {sink!r}")
+        self.sink = sink
+        self.query_heat = (float(query_heat[0]), int(query_heat[1])) if query_heat is not None else None
+        if self.query_heat is not None and self.query_heat[1] < 1:
+            raise ValueError("query_heat: 'every' must be at least one position")
+        self.head_factor = bool(head_factor)
+        self.softcap = float(softcap)
+        if self.softcap < 0:
+            raise ValueError("softcap must not be negative")
+        self.distance_slopes = bool(distance_slopes)
+        self.head_gate = bool(head_gate)
+        if value_mix not in (None, "keep", "blend"):
+            raise ValueError(f"value_mix must be None, 'keep' or 'blend', got {value_mix!r}")
+        self.value_mix = value_mix
         self.projection_float32 = bool(projection_float32)
         self.position = build_part("position", position) if position is not None else None
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(self.head_dim)
@@ -95,8 +125,8 @@ class Attention(Mixer):
         self.v_width = self.num_kv_heads * self.value_dim
         self.out_width = self.num_heads * self.value_dim
         self.qkv_width = self.q_width + self.kv_width + self.v_width
-        if qk_norm not in (None, "projection", "head"):
-            raise ValueError(f"qk_norm must be None, 'projection' or 'head', got {qk_norm!r}")
+        if qk_norm not in (None, "projection", "head", "unit"):
+            raise ValueError(f"qk_norm must be None, 'projection', 'head' or 'unit', got {qk_norm!r}")
         self.qk_norm = qk_norm
         self.value_norm = bool(value_norm)
         self.distance_penalty = bool(distance_penalty)
@@ -104,15 +134,21 @@ class Attention(Mixer):
         # the options that the rotary kernels and the tensor-core attention kernels do not know
         self.general = bool(self.qk_norm or self.value_norm or self.distance_penalty
                             or self.value_dim != self.head_dim or self.keep_first or self.gate or self.sink
-                            or self.projection_float32)
+                            or self.projection_float32 or self.query_heat or self.head_factor or self.softcap
+                            or self.distance_slopes or self.head_gate or self.value_mix)
+        if (self.head_gate or self.value_mix) and not self.projection_float32:
+            raise ValueError("a gate per head and mixed values are built for a float32 projection")
         if not self.general and (getattr(self.position, "magnitude", 1.0) != 1.0
                                  or getattr(self.position, "keep_pairing", False)):
             raise ValueError("the fused rotary kernels rotate without a magnitude factor and pair (j, j + R/2) only")
-        if self.gate and self.qkv_bias:
+        if (self.gate or self.head_gate) and self.qkv_bias:
             raise ValueError("the output gate is built for projections without biases")
+        if self.gate and self.head_gate:
+            raise ValueError("one output gate: per element or per head")
+        self.gate_width = self.out_width if self.gate else (self.num_heads if self.head_gate else 0)
         self.names = {key: key for key in ("q_proj.weight", "k_proj.weight", "v_proj.weight", "o_proj.weight",
                                            "q_proj.bias", "k_proj.bias", "v_proj.bias", "q_norm", "k_norm",
-                                           "r1", "r2", "gate", "sink")}
+                                           "r1", "r2", "gate", "sink", "factor", "value_mix")}
         self.names.update(names or {})
         self.tiled = False      # set at bind: whether prompt portions run on the tensor-core kernel
 
@@ -143,13 +179,17 @@ class Attention(Mixer):
             specs[n["q_proj.bias"]] = TensorSpec((self.q_width,), role="vector")
             specs[n["k_proj.bias"]] = TensorSpec((self.kv_width,), role="vector")
             specs[n["v_proj.bias"]] = TensorSpec((self.v_width,), role="vector")
-        if self.qk_norm:
+        if self.qk_norm in ("projection", "head"):
             per_head = self.qk_norm == "head"
             specs[n["q_norm"]] = TensorSpec((self.head_dim if per_head else self.q_width,), init="gain", role="vector")
             specs[n["k_norm"]] = TensorSpec((self.head_dim if per_head else self.kv_width,), init="gain", role="vector")
-        if self.gate:
-            specs[n["gate"]] = TensorSpec((self.out_width, self.hidden_size))
-        if self.sink:
+        if self.gate_width:
+            specs[n["gate"]] = TensorSpec((self.gate_width, self.hidden_size))
+        if self.head_factor:
+            specs[n["factor"]] = TensorSpec((self.num_heads,), init="gain", role="vector")
+        if self.value_mix:
+            specs[n["value_mix"]] = TensorSpec((), role="vector")
+        if self.sink is True:
             specs[n["sink"]] = TensorSpec((self.num_heads,), role="vector")
         if self.distance_penalty:
             specs[n["r1"]] = TensorSpec((self.num_heads,), init="gain", role="vector")
@@ -185,7 +225,7 @@ class Attention(Mixer):
             if self.paired:
                 q = ops.pair_rotary_rows(q, self.num_heads, self.head_dim, rotary)
                 k = ops.pair_rotary_rows(k, self.num_kv_heads, self.head_dim, rotary)
-            if self.gate and suffix == "weight":
+            if self.gate_width and suffix == "weight":
                 return torch.cat([q, k, v, tensors[self.names["gate"]]]).contiguous()
             return torch.cat([q, k, v]).contiguous()
 
@@ -202,16 +242,25 @@ class Attention(Mixer):
                 self.rotation = SimpleNamespace(
                     inv_freq=inv_freq.to(runtime.device).contiguous(), magnitude=self.position.magnitude,
                     interleaved=self.position.pairing == "interleaved", dims=self.position.rotary_dim)
-        self.sinks = tensors[self.names["sink"]].contiguous() if self.sink else None
-        self.q_gain = tensors[self.names["q_norm"]].contiguous() if self.qk_norm else None
-        self.k_gain = tensors[self.names["k_norm"]].contiguous() if self.qk_norm else None
+        self.sinks = tensors[self.names["sink"]].contiguous() if self.sink is True else None
+        if self.sink == "one":
+            self.sinks = torch.zeros(self.num_heads, dtype=torch.float32, device=runtime.device)
+        gained = self.qk_norm in ("projection", "head")
+        self.q_gain = tensors[self.names["q_norm"]].contiguous() if gained else None
+        self.k_gain = tensors[self.names["k_norm"]].contiguous() if gained else None
+        self.factor = tensors[self.names["factor"]].contiguous() if self.head_factor else None
+        self.value_share = tensors[self.names["value_mix"]].reshape(1).contiguous() if self.value_mix == "blend" else None
+        self.slopes = None
+        if self.distance_slopes:
+            slopes = [2.0 ** (-8.0 * (h + 1) / self.num_heads) for h in range(self.num_heads)]
+            self.slopes = torch.tensor(slopes, dtype=torch.float64).to(device=runtime.device, dtype=torch.float32)
         self.distance = ((tensors[self.names["r1"]].contiguous(), tensors[self.names["r2"]].contiguous())
                          if self.distance_penalty else None)
-        # the tensor-core kernels take bfloat16 heads of a multiple of 16 elements, values as large as keys
-        self.tiled = bool(self.value_dim == self.head_dim and self.head_dim % 16 == 0 and self.head_dim <= 256
+        # the tensor-core kernels take bfloat16 heads of a multiple of 16 elements, keys and values alike or not
+        self.tiled = bool(self.value_dim % 16 == 0 and self.head_dim % 16 == 0 and max(self.head_dim, self.value_dim) <= 256
                           and runtime.dtype_name == "bfloat16")
         if not self.general or self.tiled:
-            runtime.ops.require_attention(self.head_dim)
+            runtime.ops.require_attention(max(self.head_dim, self.value_dim))
 
     takes_normed_input = True   # x goes to ops.linear only
     kernels_through_ops = True  # every kernel of this part is a method of ``Ops``: a decode step may be recorded
@@ -224,7 +273,7 @@ class Attention(Mixer):
         rt = self.runtime
         tokens = x.shape[0]
         kv = binding.kv
-        width = self.qkv_width + (self.out_width if self.gate else 0)
+        width = self.qkv_width + self.gate_width
         if self.projection_float32:
             qkv = rt.workspace.get("attention.qkv32", tokens, width, torch.float32)
             qkv = rt.ops.linear(x, self.w_qkv, self.b_qkv, qkv)
@@ -232,14 +281,17 @@ class Attention(Mixer):
             qkv = rt.workspace.get("attention.qkv", tokens, width, rt.dtype)
             qkv = rt.ops.linear(x, self.w_qkv, self.b_qkv, qkv, tag="attention.qkv", defer_bias=True)
         q = rt.workspace.get("attention.q", tokens, self.q_width, rt.dtype)
+        kept = rt.workspace.get("attention.kept_values", tokens, self.v_width, torch.float32) if self.value_mix else None
         rt.ops.norm_kv_write(qkv, ctx, kv, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim,
                              self.q_gain, self.k_gain, self.value_norm, self.norm_eps, q,
                              write_cache=binding.owns_cache, per_head=self.qk_norm == "head",
-                             rotation=self.rotation)
+                             rotation=self.rotation, unit_heads=self.qk_norm == "unit", q_factor=self.factor,
+                             heat=self.query_heat, first_values=kept, value_share=self.value_share)
         mixed = rt.workspace.get("attention.out", tokens, self.out_width, rt.dtype)
         rt.ops.attention_penalised(q, mixed, ctx, kv, self.num_heads, self.num_kv_heads, self.head_dim,
                                    self.value_dim, self.scale, self.window, self.distance,
-                                   keep_first=self.keep_first, sinks=self.sinks)
+                                   keep_first=self.keep_first, sinks=self.sinks, softcap=self.softcap,
+                                   slopes=self.slopes, gates=qkv[:, self.qkv_width:] if self.head_gate else None)
         if self.gate:
             if self.projection_float32:
                 raise ValueError("the output gate reads a projection of the compute dtype")

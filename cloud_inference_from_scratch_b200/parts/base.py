@@ -97,6 +97,13 @@ class Part:
     def bind(self, tensors: dict[str, "torch.Tensor"], runtime: "Runtime") -> None:
         self.runtime = runtime
 
+    def shared_tensor_specs(self) -> dict[str, TensorSpec]:
+        """Tensors that several layers read, by their full names in the weight files (no prefix)."""
+        return {}
+
+    def bind_shared(self, tensors: dict[str, "torch.Tensor"]) -> None:
+        """Takes the shared tensors (one copy on the device for all layers), after ``bind``."""
+
     def subparts(self) -> "tuple[Part, ...]":
         """Parts this part is put together from (a mixer made of two mixers names them here), for whoever walks
         all parts of a model: the step function looking for planners, for instance."""

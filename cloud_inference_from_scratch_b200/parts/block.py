@@ -12,7 +12,10 @@ from .base import Block, register_part
 
 def _normalise(norm, consumer, residual, pending, ctx):
     """A consumer that declares ``takes_normed_input`` may get the norm un-computed (see
-    ``Norm.forward_lazy``); every other pairing runs the norm's kernel."""
+    ``Norm.forward_lazy``), one that declares ``takes_pending_norm`` gets it not even begun; every other pairing
+    runs the norm's kernel."""
+    if getattr(consumer, "takes_pending_norm", False) and hasattr(norm, "forward_pending"):
+        return norm.forward_pending(residual, pending, ctx)
     lazy = getattr(norm, "forward_lazy", None)
     if lazy is not None and getattr(consumer, "takes_normed_input", False):
         return lazy(residual, pending, ctx)
@@ -27,7 +30,9 @@ def _lazy_gain(norm, consumer):
 
 
 class PreNormResidual(Block):
-    """``feed_forward`` and ``feed_forward_norm`` may both be left out: the layer is then its mixer sublayer alone."""
+    """``feed_forward`` and ``feed_forward_norm`` may both be left out: the layer is then its mixer sublayer alone.
+    A ``side`` part, if there is one, comes last: it reads the stream itself (no norm), with the pending update,
+    and returns an update of its own."""
 
     slots = ("mixer", "mixer_norm")
     kernels_through_ops = True   # the block itself launches nothing
@@ -48,6 +53,10 @@ class PreNormResidual(Block):
             # the next layer's first) or a norm kernel: before their dependency wait they ask for
             # weights only, so the projection may let them start early
             sink.early_trigger = True
+        side = self.parts.get("side")
+        if side is not None:
+            update = self._sublayers(residual, pending, ctx, binding)
+            return side.forward_stream(residual, update, ctx)
         x = _normalise(self.mixer_norm, self.mixer, residual, pending, ctx)
         if not self.has_feed_forward:
             if sink is not None:   # the mixer's sum is read next by whoever comes after this layer
@@ -60,6 +69,17 @@ class PreNormResidual(Block):
         if sink is not None:   # the feed-forward's sum by whoever comes after this layer
             sink.gain = sink.following_gain
         return self.feed_forward.forward(x, ctx)
+
+    def _sublayers(self, residual, pending, ctx, binding):
+        """The sublayers of a layer with a ``side`` part, none of which adds itself into the stream."""
+        sink = getattr(ctx, "residual_sink", None)
+        ctx.residual_sink = None
+        update = self.mixer.forward(_normalise(self.mixer_norm, self.mixer, residual, pending, ctx), ctx, binding)
+        if self.has_feed_forward:
+            update = self.feed_forward.forward(
+                _normalise(self.feed_forward_norm, self.feed_forward, residual, update, ctx), ctx)
+        ctx.residual_sink = sink
+        return update
 
 
 register_part("block", "prenorm_residual", PreNormResidual, replace=True)

@@ -8,7 +8,7 @@ the same kernel, and the result is rounded once to the compute dtype.
 
 from __future__ import annotations
 
-from ..lazy import Accumulated, NormedInput
+from ..lazy import Accumulated, NormedInput, PendingNorm
 from .base import Norm, TensorSpec, register_part
 
 
@@ -136,3 +136,47 @@ class StreamRMSNorm(Norm):
 
 
 register_part("norm", "stream_rmsnorm", StreamRMSNorm, replace=True)
+
+
+class GroupRMSNorm(Norm):
+    """RMS norm of a row in ``groups`` equal consecutive parts, each divided by its OWN root mean square
+    (``x / sqrt(mean(x^2) + eps)`` over the part), the whole multiplied by a gain vector [H]; fused with the pending
+    residual add, which may itself be a ``NormedUpdate``.  One group is the ordinary RMS norm.  ``name``: the tensor's
+    name after the part's prefix."""
+
+    kernels_through_ops = True
+
+    def __init__(self, hidden_size: int, eps: float, groups: int = 1, name: str = "weight") -> None:
+        if groups < 1 or hidden_size % groups:
+            raise ValueError(f"a row of {hidden_size} does not divide into {groups} groups")
+        self.hidden_size = int(hidden_size)
+        self.eps = float(eps)
+        self.groups = int(groups)
+        self.name = str(name)
+
+    def tensor_specs(self) -> dict[str, TensorSpec]:
+        return {self.name: TensorSpec((self.hidden_size,), init="gain", role="vector")}
+
+    def bind(self, tensors, runtime) -> None:
+        self.runtime = runtime
+        runtime.ops.require_grouped()
+        self.weight = tensors[self.name].contiguous()
+
+    def forward(self, residual, update, ctx, rows=None):
+        rt = self.runtime
+        count = residual.shape[0] if rows is None else rows.shape[0]
+        out = rt.workspace.get("norm.out" if rows is None else "norm.rows", count,
+                               self.hidden_size, rt.dtype, per_request=rows is not None)
+        rt.ops.group_norm(residual, update, self.weight, self.eps, self.groups, out, rows)
+        return out
+
+    def forward_pending(self, residual, update, ctx):
+        """For a consumer whose own kernel begins with this norm (``takes_pending_norm``): nothing runs here."""
+        return PendingNorm(residual, update, self.weight, self.eps, self.groups)
+
+    def normalise_stream(self, residual) -> None:
+        """The float32 stream itself becomes its norm (a model that normalises its embedding rows)."""
+        self.runtime.ops.group_norm(residual, None, self.weight, self.eps, self.groups, residual)
+
+
+register_part("norm", "group_rmsnorm", GroupRMSNorm, replace=True)

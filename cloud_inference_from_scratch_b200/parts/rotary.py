@@ -24,6 +24,9 @@ Beyond the reference (which has exactly the above):
   ``f_i / factor * r_i + f_i * (1 - r_i)``; cos and sin are then both multiplied by
   ``magnitude = 0.1 ln(factor) + 1`` (a mixer that rotates with kernels of its own reads
   ``magnitude``; the softmax scale is left alone).
+* ``bands`` = (factor, low, high, original) scales frequencies by wavelength: with ``l = 2 pi / f``, f stays where
+  ``l < original / high``, becomes ``f / factor`` where ``l > original / low``, and between the two, with
+  ``s = (original / l - low) / (high - low)``, ``(1 - s) f / factor + s f``; no magnitude factor.
 * ``keep_pairing``: ``row_order`` answers None although the pairing is interleaved, for a mixer whose
   kernels rotate either pairing themselves (``pairing`` tells them which).
 """
@@ -40,7 +43,8 @@ class RopeNeox(PositionEncoding):
 
     def __init__(self, head_dim: int, rotary_dim: int, theta: float, max_positions: int,
                  pairing: str = "half", position_scale: float = 1.0, attention_factor: float = 1.0,
-                 ramp: tuple[float, float, float, float] | None = None, keep_pairing: bool = False) -> None:
+                 ramp: tuple[float, float, float, float] | None = None, keep_pairing: bool = False,
+                 bands: tuple[float, float, float, float] | None = None) -> None:
         if rotary_dim % 2 or rotary_dim > head_dim or rotary_dim < 2:
             raise ValueError(f"rotary_dim {rotary_dim} must be even and within head_dim {head_dim}")
         if pairing not in ("half", "interleaved"):
@@ -59,11 +63,27 @@ class RopeNeox(PositionEncoding):
             raise ValueError("ramp must be (factor, original, fast, slow), all positive")
         self.magnitude = 0.1 * math.log(self.ramp[0]) + 1.0 if self.ramp is not None else 1.0
         self.keep_pairing = bool(keep_pairing)
+        self.bands = tuple(float(value) for value in bands) if bands is not None else None
+        if self.bands is not None and (len(self.bands) != 4 or min(self.bands) <= 0 or self.ramp is not None):
+            raise ValueError("bands must be (factor, low, high, original), all positive, and exclude a ramp")
 
     def frequencies(self) -> list[float]:
         """f_i for i < rotary_dim / 2, in double precision."""
         dims, half = self.rotary_dim, self.rotary_dim // 2
         plain = [self.theta ** (-2.0 * i / dims) / self.position_scale for i in range(half)]
+        if self.bands is not None:
+            factor, low, high, original = self.bands
+
+            def banded(f: float) -> float:
+                turns = original * f / (2.0 * math.pi)          # original / wavelength
+                if turns > high:
+                    return f
+                if turns < low:
+                    return f / factor
+                s = (turns - low) / (high - low) if high != low else 1.0
+                return (1.0 - s) * f / factor + s * f
+
+            return [banded(f) for f in plain]
         if self.ramp is None:
             return plain
         factor, original, fast, slow = self.ramp
@@ -90,7 +110,7 @@ class RopeNeox(PositionEncoding):
         import torch
 
         self.runtime = runtime
-        if self.ramp is None:
+        if self.ramp is None and self.bands is None:
             exponent = torch.arange(0, self.rotary_dim, 2, dtype=torch.float32) / self.rotary_dim
             inv_freq = 1.0 / (self.theta ** exponent) / self.position_scale
         else:

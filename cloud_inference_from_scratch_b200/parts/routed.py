@@ -13,7 +13,11 @@ interleaved in blocks of 16);
 Two options: ``router_bias`` adds a stored vector to the logits, and ``score="chosen_softmax"`` chooses the
 experts with the largest logits and weights them by the softmax over the chosen logits alone.
 
-the kernels group the (token, expert) pairs by expert on the device and never tell the host how
+``score="sigmoid"`` makes the scores sigmoids of the logits.  ``groups`` = (count, keep): the experts form ``count``
+equal groups of neighbours, a group's score is the sum of its two largest choice scores (score + correction), and only
+experts of the ``keep`` best groups can be chosen.  ``norm_floor`` is added to the sum that ``renormalize`` divides by.
+
+The kernels group the (token, expert) pairs by expert on the device and never tell the host how
 many tokens an expert got, so a step is one fixed sequence of launches.
 """
 
@@ -25,7 +29,8 @@ from .base import FeedForward, TensorSpec, register_part
 class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, intermediate_size: int, num_experts: int, top: int,
                  correction: bool = True, renormalize: bool = False,
-                 names: dict[str, str] | None = None, router_bias: bool = False, score: str = "softmax") -> None:
+                 names: dict[str, str] | None = None, router_bias: bool = False, score: str = "softmax",
+                 groups: tuple[int, int] = (1, 1), norm_floor: float = 0.0) -> None:
         if not 1 <= top <= num_experts:
             raise ValueError("top must lie in 1..num_experts")
         self.hidden_size = int(hidden_size)
@@ -35,8 +40,15 @@ class RoutedExperts(FeedForward):
         self.correction = bool(correction)
         self.renormalize = bool(renormalize)
         self.router_bias = bool(router_bias)
-        if score not in ("softmax", "chosen_softmax"):
-            raise ValueError(f"routed experts: score {score!r} is not built (known: softmax, chosen_softmax)")
+        if score not in ("softmax", "chosen_softmax", "sigmoid"):
+            raise ValueError(f"routed experts: score {score!r} is not built (known: softmax, chosen_softmax, sigmoid)")
+        count, keep = (int(number) for number in groups)
+        if count < 1 or num_experts % count or not 1 <= keep <= count or top > num_experts // count * keep:
+            raise ValueError(f"routed experts: {keep} of {count} groups of {num_experts} experts cannot give {top} choices")
+        if count > 1 and score == "chosen_softmax":
+            raise ValueError("routed experts: groups are built for a choice among scores, not among logits")
+        self.groups = (count, keep)
+        self.norm_floor = float(norm_floor)
         if score == "chosen_softmax" and correction:
             raise ValueError("routed experts: a correction steers a choice among softmax scores, not among logits")
         self.score = score
@@ -81,7 +93,8 @@ class RoutedExperts(FeedForward):
         update = rt.workspace.get("feed_forward.update32", x.shape[0], self.hidden_size, torch.float32)
         return rt.ops.routed_experts(x, self.router, self.bias, self.w_gate, self.w_up, self.w_down,
                                      self.top, self.renormalize, update, rt.workspace, router_bias=self.logit_bias,
-                                     chosen_softmax=self.score == "chosen_softmax")
+                                     chosen_softmax=self.score == "chosen_softmax",
+                                     sigmoid=self.score == "sigmoid", groups=self.groups, norm_floor=self.norm_floor)
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts, replace=True)
