@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200, random weights.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl own|reference]
-                    [--config 3b|7b-mixed|14b-pressure|zisesun|lodalix|lazilorn|bilipel] [--quick]
+                    [--config 3b|7b-mixed|14b-pressure|zisesun|lodalix|lazilorn|bilipel|sutuvik] [--quick]
 
 Prints ONE JSON line.  The default configuration is the Qwen2.5-3B shape: a "step" is one decode
 step of a batch of requests whose prompts (2,048 random tokens each) were prefilled before;
@@ -42,6 +42,12 @@ of 256 and 512 tokens, and (unless ``--quick``) the two other benchmark configur
   channel; a gated dense feed-forward or routed experts; layer norms; looped layers) at two sizes, beside the
   Qwen2 dense shape of equal width, layer runs, head count and active feed-forward size and beside the Lodalix
   configuration of that size, measured the same way.
+
+* ``sutuvik``: the Sutuvik design (Mamba-2; softmax attention without rotation, with a query temperature, slopes, a
+  sink and a gate per head; softmax attention with rotation before a norm, factors per head, a soft cap and one in the
+  denominator; mixed values; an input convolution in front of every mixer; experts chosen from the best groups; a
+  token side input) at two sizes, beside the Qwen2 dense shape of equal width, layer count, head count and active
+  feed-forward size and beside the Zisesun configuration of that size, measured the same way.
 
 ``check`` compares, at the full 36 layers, the logits of the bfloat16 generation path with the
 32-bit path of the same weights (``engine/check.py``).  ``--config`` prints the line of one of the
@@ -681,7 +687,31 @@ BILIPEL_SIZES = {
     "w4096": (_bilipel(4096, "ALG", (2, 3, 2), 32, 8, 128, 64, 512, 1024, 32, 8192, 32, 4, 2048),
               dict(_qwen2(4096, 4, 32, 8, 8192, 32000, False)), LODALIX_SIZES["w4096"][0]),
 }
-NEAREST_DESIGN = {"lazilorn": "zisesun", "bilipel": "lodalix"}
+
+
+def _sutuvik(width, layers, heads, kv_heads, dim, mamba_heads, vdim, state, experts, top, ff, side, vocab=32000) -> dict:
+    """``layers``: a string of B (attention with slopes, a sink and a gate per head), R (rotated attention with a soft
+    cap) and M (Mamba-2), routed experts in every layer."""
+    mlp = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=experts, top=top, groups=dict(count=4, keep=2)))
+    sizes = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, v_mix=True)
+    rot = dict(base=500000.0, dims=dim, scaling=dict(factor=4.0, low=1.0, high=4.0, original=1024))
+    kinds = {
+        "B": dict(type="attention", mixer=dict(sizes, q_temp=dict(coef=0.1, every=1024)), mlp=mlp),
+        "R": dict(type="attention_2", mixer=dict(sizes, scale=dim ** 0.5 / 4, softcap=30.0, rot=rot), mlp=mlp),
+        "M": dict(type="mamba2", mixer=dict(heads=mamba_heads, vdim=vdim, state=state, groups=1, conv=4, norm_groups=4), mlp=mlp),
+    }
+    return dict(architecture="Sutuvik", vocab=vocab, width=width, logit_scale=0.25, norm=dict(eps=1e-6, groups=4),
+                canon=dict(taps=4), token_side=dict(dim=side), layers=[kinds[letter] for letter in layers])
+
+
+# (Sutuvik configuration, the Qwen2 dense shape of equal width, layers, heads and ACTIVE feed-forward size, and the
+# Zisesun configuration of that size: the design whose parts are nearest, attention with a distance penalty, a float32
+# matrix recurrence with one decay a head and routed experts in every layer)
+SUTUVIK_SIZES = {
+    "w2048": (_sutuvik(2048, "RMBMRMBM", 16, 2, 128, 64, 64, 128, 16, 4, 1376, 128), *ZISESUN_SIZES["w2048"][::-1]),
+    "w4096": (_sutuvik(4096, "RMBM", 32, 8, 128, 128, 64, 128, 32, 4, 2048, 256), *ZISESUN_SIZES["w4096"][::-1]),
+}
+NEAREST_DESIGN = {"lazilorn": "zisesun", "bilipel": "lodalix", "sutuvik": "zisesun"}
 
 
 def _time_step_function(cfg: dict, batch: int, steps: int, warmup: int, only: str = "all") -> dict:
@@ -756,7 +786,7 @@ def run_design(args: argparse.Namespace, design: str = "zisesun") -> int:
     import torch
 
     sizes = {"zisesun": ZISESUN_SIZES, "lodalix": LODALIX_SIZES, "lazilorn": LAZILORN_SIZES,
-             "bilipel": BILIPEL_SIZES}[design]
+             "bilipel": BILIPEL_SIZES, "sutuvik": SUTUVIK_SIZES}[design]
     near = NEAREST_DESIGN.get(design)
     title = design.capitalize()
 
@@ -775,6 +805,7 @@ def run_design(args: argparse.Namespace, design: str = "zisesun") -> int:
         if args.layers:
             zisesun = dict(zisesun, layers=zisesun["layers"][:args.layers])
             qwen = dict(qwen, num_hidden_layers=args.layers)
+            nearest = [dict(other, layers=other["layers"][:args.layers]) for other in nearest]
         points[name] = {}
         if args.model in ("both", design):
             points[name][design] = _time_step_function(zisesun, args.batch, args.steps, args.warmup, args.only)
@@ -831,12 +862,12 @@ def main() -> int:
                              "default is 2048; longer ones are for profiles of long contexts, own arm only)")
     parser.add_argument("--impl", default="own", choices=("own", "reference"))
     parser.add_argument("--size", default="all", help="--config zisesun or lodalix: one of its sizes (w2048, w4096)")
-    parser.add_argument("--model", default="both", choices=("both", "zisesun", "lodalix", "lazilorn", "bilipel", "qwen2"),
-                        help="--config zisesun, lodalix, lazilorn or bilipel: only that design, or only its dense peer "
-                             "(--config lazilorn --model zisesun, --config bilipel --model lodalix: only the nearest "
+    parser.add_argument("--model", default="both", choices=("both", "zisesun", "lodalix", "lazilorn", "bilipel", "sutuvik", "qwen2"),
+                        help="--config zisesun, lodalix, lazilorn, bilipel or sutuvik: only that design, or only its dense peer "
+                             "(--config lazilorn or sutuvik --model zisesun, --config bilipel --model lodalix: only the nearest "
                              "design's configuration of that size)")
     parser.add_argument("--config", default="3b",
-                        choices=("3b", "7b-mixed", "14b-pressure", "zisesun", "lodalix", "lazilorn", "bilipel"),
+                        choices=("3b", "7b-mixed", "14b-pressure", "zisesun", "lodalix", "lazilorn", "bilipel", "sutuvik"),
                         help="the benchmark configuration whose line is printed (default: the 3B line, "
                              "which also carries the other two as points)")
     parser.add_argument("--quick", action="store_true",
@@ -860,7 +891,7 @@ def main() -> int:
         CONTEXT = min(limit, PROMPT_TOKENS + max(2048, room))
     if args.impl == "reference":
         return run_reference(args)
-    if args.config in ("zisesun", "lodalix", "lazilorn", "bilipel"):
+    if args.config in ("zisesun", "lodalix", "lazilorn", "bilipel", "sutuvik"):
         return run_design(args, args.config)
     if args.config != "3b":
         return run_other_config(args)

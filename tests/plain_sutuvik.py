@@ -15,6 +15,15 @@ import torch
 F64 = torch.float64
 
 
+NOISE = [None]      # a generator: what a 16-bit engine rounds (inputs of products, cached rows) is moved about as much
+
+
+def rounded(x):
+    if NOISE[0] is None:
+        return x
+    return x * (1.0 + (torch.rand(x.shape, generator=NOISE[0], dtype=F64) - 0.5) * 2.0 ** -8)
+
+
 def rms(x, eps):
     return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
 
@@ -130,9 +139,9 @@ def biased_mixer(h, w, m, eps, carry):
     v = mix_values((h @ w["v"].T).view(tokens, groups, m["vdim"]), w, m, carry)
     heat = m["q_temp"]
     q = q * query_temperature(torch.arange(tokens), heat["coef"], heat["every"]).view(-1, 1, 1)
-    o = attend(q, k, v, m["scale"], w["sink"], slopes=head_slopes(heads))
+    o = attend(rounded(q), rounded(k), rounded(v), m["scale"], w["sink"], slopes=head_slopes(heads))
     o = o * torch.sigmoid(h @ w["g"].T).unsqueeze(-1)
-    return o.reshape(tokens, -1) @ w["o"].T
+    return rounded(o.reshape(tokens, -1)) @ w["o"].T
 
 
 def rotated_mixer(h, w, m, eps, carry):
@@ -142,8 +151,8 @@ def rotated_mixer(h, w, m, eps, carry):
     q = rms(rotate_pairs((h @ w["q"].T).view(tokens, heads, m["dim"]), at, m["rot"]), eps)
     k = rms(rotate_pairs((h @ w["k"].T).view(tokens, groups, m["dim"]), at, m["rot"]), eps)
     v = mix_values((h @ w["v"].T).view(tokens, groups, m["vdim"]), w, m, carry)
-    o = attend(q, k, v, m["scale"], torch.zeros(heads, dtype=F64), temps=w["temp"], cap=m["softcap"])
-    return o.reshape(tokens, -1) @ w["o"].T
+    o = attend(rounded(q), rounded(k), rounded(v), m["scale"], torch.zeros(heads, dtype=F64), temps=w["temp"], cap=m["softcap"])
+    return rounded(o.reshape(tokens, -1)) @ w["o"].T
 
 
 def state_space(x, b, c, dt, a_log, d, state=None):
@@ -172,7 +181,7 @@ def mamba_mixer(h, w, m, eps, carry):
     y, _ = state_space(x.reshape(tokens, heads, vdim), b.reshape(tokens, groups, n), c.reshape(tokens, groups, n), dt,
                        w["A_log"], w["D"])
     y = group_norm(y.reshape(tokens, inner) * silu(z), w["norm"], eps, m["norm_groups"])
-    return y @ w["o"].T
+    return rounded(y) @ w["o"].T
 
 
 def choose_experts(h, w, router):
@@ -196,13 +205,13 @@ def routed_feed_forward(h, w, mlp):
         rows, slots = torch.where(ids == expert)
         if rows.numel():
             e = f"e{expert}."
-            y = (silu(h[rows] @ w[e + "gate"].T) * (h[rows] @ w[e + "up"].T)) @ w[e + "down"].T
+            y = rounded(silu(h[rows] @ w[e + "gate"].T) * (h[rows] @ w[e + "up"].T)) @ w[e + "down"].T
             out[rows] += share[rows, slots].unsqueeze(-1) * y
     return out
 
 
 def token_side(x, e, w, eps):
-    y = (gelu_tanh(x @ w["side.gate"].T) * e) @ w["side.proj"].T
+    y = rounded(gelu_tanh(rounded(x) @ w["side.gate"].T) * e) @ w["side.proj"].T
     return x + rms(y, eps) * w["side.norm"]
 
 
@@ -211,11 +220,6 @@ MIXERS = {"mamba2": mamba_mixer, "attention": biased_mixer, "attention_2": rotat
 
 def sub(weights, prefix):
     return {name[len(prefix):]: tensor.to(F64) for name, tensor in weights.items() if name.startswith(prefix)}
-
-
-def rounded(h, on):
-    """The sublayer's input as a bfloat16 product would see it (``on``), or as it is."""
-    return h.to(torch.bfloat16).to(F64) if on else h
 
 
 def read_folder(folder):
@@ -238,9 +242,18 @@ def greedy(config, weights, prompt, count):
     return tokens[len(prompt):]
 
 
-def forward(config, weights, tokens, streams=None, round_inputs=False):
+def forward(config, weights, tokens, streams=None, noise=None):
     """Logits [T, vocab] of one sequence in float64.  ``streams``: a list that receives the stream after every
-    layer.  ``round_inputs``: every sublayer reads its input rounded to bfloat16 (everything else stays exact)."""
+    layer.  ``noise``: a seed; inputs of products and rows that a cache holds are then each moved by up to the rounding
+    of bfloat16 (everything else stays exact)."""
+    NOISE[0] = None if noise is None else torch.Generator().manual_seed(noise)
+    try:
+        return _forward(config, weights, tokens, streams)
+    finally:
+        NOISE[0] = None
+
+
+def _forward(config, weights, tokens, streams):
     eps, groups = config["norm"]["eps"], config["norm"]["groups"]
     w = {name: tensor.to(F64) for name, tensor in weights.items()}
     ids = torch.as_tensor(tokens, dtype=torch.long)
@@ -250,12 +263,11 @@ def forward(config, weights, tokens, streams=None, round_inputs=False):
     for index, layer in enumerate(config["layers"]):
         lw = sub(w, f"l{index}.")
         h = group_norm(x, lw["norm1"], eps, groups)
-        h = rounded(h + causal_conv(h, lw["canon1"]), round_inputs)
+        h = rounded(h + causal_conv(h, lw["canon1"]))
         x = x + MIXERS[layer["type"]](h, sub(lw, "mix."), layer["mixer"], eps, carry)
         if layer.get("mlp"):
-            x = x + routed_feed_forward(rounded(group_norm(x, lw["norm2"], eps, groups), round_inputs), sub(lw, "mlp."),
-                                        layer["mlp"])
+            x = x + routed_feed_forward(rounded(group_norm(x, lw["norm2"], eps, groups)), sub(lw, "mlp."), layer["mlp"])
         x = token_side(x, side[:, index * dim:(index + 1) * dim], lw, eps)
         if streams is not None:
             streams.append(x)
-    return group_norm(x, w["final.norm"], eps, groups) @ w["embed"].T * config["logit_scale"]
+    return rounded(group_norm(x, w["final.norm"], eps, groups)) @ w["embed"].T * config["logit_scale"]
