@@ -185,6 +185,68 @@ __global__ void short_conv_kernel(const float* __restrict__ proj, int proj_strid
   out[(size_t)t * out_stride + c] = acc / (1.f + expf(-acc));
 }
 
+// The same for prompt portions: four channels a thread (16-byte pieces), the filter in registers, kConvRun tokens a
+// thread one after the other, so that a row is read from memory once and then found in the cache.
+constexpr int kConvRun = 8, kConvThreads = 128;
+template <int TAPS>
+__global__ void __launch_bounds__(kConvThreads)
+short_conv_run_kernel(const float* __restrict__ proj, int proj_stride, const float* __restrict__ w,
+                      const float* __restrict__ bias, const float* __restrict__ state, long long state_stride,
+                      float* __restrict__ out, int out_stride, const int* __restrict__ query_start,
+                      const int* __restrict__ request_of_token, const int* __restrict__ slots, int tokens, int channels,
+                      int max_slots, int* err) {
+  pdl_wait();
+  pdl_trigger();
+  const int c = (blockIdx.y * kConvThreads + threadIdx.x) * 4;
+  if (c >= channels) return;
+  float f[4][TAPS], b[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    b[e] = bias ? bias[c + e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) f[e][j] = w[(size_t)(c + e) * TAPS + j];
+  }
+  const int t0 = blockIdx.x * kConvRun, t1 = min(t0 + kConvRun, tokens);
+  float4 window[TAPS];          // the inputs of the last TAPS tokens of the request
+  int request = -1, begin = 0;
+  for (int t = t0; t < t1; ++t) {
+    const int r = request_of_token[t];
+    if (r != request) {           // the run's first token, or another request's: fill the window
+      request = r;
+      begin = query_start[r];
+      const int slot = slots[r];
+      if (slot < 0 || slot >= max_slots) {
+        atomicOr(err, kErrBadRequest);
+        return;
+      }
+      const float* hist = state + (size_t)slot * state_stride;
+#pragma unroll
+      for (int j = 1; j < TAPS; ++j) {
+        const int src = t - begin - (TAPS - j);
+        window[j] = src >= 0 ? *reinterpret_cast<const float4*>(proj + (size_t)(begin + src) * proj_stride + c)
+                             : *reinterpret_cast<const float4*>(hist + (size_t)(TAPS - 1 + src) * channels + c);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j) window[j] = window[j + 1];
+    window[TAPS - 1] = *reinterpret_cast<const float4*>(proj + (size_t)t * proj_stride + c);
+    float acc[4] = {};
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      acc[0] = fmaf(f[0][j], window[j].x, acc[0]);
+      acc[1] = fmaf(f[1][j], window[j].y, acc[1]);
+      acc[2] = fmaf(f[2][j], window[j].z, acc[2]);
+      acc[3] = fmaf(f[3][j], window[j].w, acc[3]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (bias) acc[e] += b[e];
+      acc[e] = acc[e] / (1.f + expf(-acc[e]));
+    }
+    *reinterpret_cast<float4*>(out + (size_t)t * out_stride + c) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+  }
+}
+
 // The same for a step of single tokens (row t is request t): a thread reads its channel's history, writes the result
 // and moves the history on.
 __global__ void short_conv_single_kernel(const float* __restrict__ proj, int proj_stride, const float* __restrict__ w,
@@ -1453,9 +1515,22 @@ extern "C" int cie_short_conv(const float* proj, int proj_stride, const float* w
                err);
     return 0;
   }
-  CIE_LAUNCH("short_conv", short_conv_kernel, dim3(tokens, blocks), dim3(threads), 0, (cudaStream_t)stream, proj,
-             proj_stride, w, bias, taps, (const float*)state, state_stride, out, out_stride, query_start, request_of_token,
-             slots, channels, max_slots, err);
+  const bool wide = channels % 4 == 0 && proj_stride % 4 == 0 && out_stride % 4 == 0 && state_stride % 4 == 0 &&
+                    ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(out) |
+                      reinterpret_cast<uintptr_t>(state)) & 15) == 0;
+  const dim3 run_grid((tokens + kConvRun - 1) / kConvRun, (channels + 4 * kConvThreads - 1) / (4 * kConvThreads));
+#define CIE_CONV_RUN(N)                                                                                             \
+  CIE_LAUNCH("short_conv", short_conv_run_kernel<N>, run_grid, dim3(kConvThreads), 0, (cudaStream_t)stream, proj,   \
+             proj_stride, w, bias, (const float*)state, state_stride, out, out_stride, query_start, request_of_token, \
+             slots, tokens, channels, max_slots, err)
+  if (wide && taps == 2) CIE_CONV_RUN(2);
+  else if (wide && taps == 3) CIE_CONV_RUN(3);
+  else if (wide && taps == 4) CIE_CONV_RUN(4);
+  else
+    CIE_LAUNCH("short_conv", short_conv_kernel, dim3(tokens, blocks), dim3(threads), 0, (cudaStream_t)stream, proj,
+               proj_stride, w, bias, taps, (const float*)state, state_stride, out, out_stride, query_start,
+               request_of_token, slots, channels, max_slots, err);
+#undef CIE_CONV_RUN
   if (taps > 1)
     CIE_LAUNCH("short_conv_keep", short_conv_keep_kernel, dim3(requests, blocks), dim3(threads), 0,
                (cudaStream_t)stream, proj, proj_stride, taps, state, state_stride, query_start, slots, request_active,

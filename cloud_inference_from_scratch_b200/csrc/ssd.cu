@@ -33,6 +33,19 @@ constexpr int kLd = kTile + 4;       // padded tile row: 16-byte pieces, few ban
 
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
+template <int V> __device__ __forceinline__ void load_v(float (&dst)[V], const float* src) {
+  if constexpr (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(src);
+    dst[0] = v.x; dst[1] = v.y; dst[2] = v.z; dst[3] = v.w;
+  } else {
+    dst[0] = src[0];
+  }
+}
+template <int V> __device__ __forceinline__ void store_v(float* dst, const float (&v)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+  else dst[0] = v[0];
+}
+
 // Columns of a float32 row: x (heads x vdim), B and C (groups x state) of `rows`; the rate of `proj`.
 struct Inputs {
   const float* rows;
@@ -115,9 +128,10 @@ ssd_scan_kernel(Inputs in, float* __restrict__ out, int out_stride, float* __res
 }
 
 // ---------------------------------------------------------------- chunks
-// grid (chunks, ceil(heads / 128)): a thread a head walks the chunk's tokens.  gates: [T][heads] pairs (dt, b).
+// grid (chunks, ceil(heads / 128)): a thread a head walks the chunk's tokens.  gates: [T][heads] pairs (dt, b); decays:
+// [chunks][heads], exp of the chunk's last b.
 __global__ void __launch_bounds__(128)
-ssd_gates_kernel(Inputs in, float2* __restrict__ gates, const int* __restrict__ chunk_row, const int* __restrict__ chunk_count) {
+ssd_gates_kernel(Inputs in, float2* __restrict__ gates, float* __restrict__ decays, const int* __restrict__ chunk_row, const int* __restrict__ chunk_count) {
   pdl_wait();
   pdl_trigger();
   const int head = blockIdx.y * 128 + threadIdx.x;
@@ -138,6 +152,7 @@ ssd_gates_kernel(Inputs in, float2* __restrict__ gates, const int* __restrict__ 
       gates[(size_t)(row0 + j0 + u) * in.heads + head] = make_float2(d, sum);
     }
   }
+  decays[(size_t)blockIdx.x * in.heads + head] = expf(sum);
 }
 
 // acc[a][b] += sum over `depth` rows of left[k][4 ty + a] * right[k][4 tx + b]
@@ -264,16 +279,18 @@ ssd_chunk_sums_kernel(Inputs in, const float2* __restrict__ gates, float* __rest
   }
 }
 
-// grid (requests, heads, blocks over state * vdim)
-__global__ void __launch_bounds__(256)
+// grid (requests, heads, blocks over state * vdim): a thread walks V neighbouring numbers of a head's state through the
+// request's chunks.  decays: [chunks][heads], what a chunk leaves of the state before it.
+template <int V>
+__global__ void __launch_bounds__(128)
 ssd_chunk_walk_kernel(float* __restrict__ sums, float* __restrict__ state, long long state_stride,
-                      const float2* __restrict__ gates, const int* __restrict__ request_chunk_start,
-                      const int* __restrict__ chunk_row, const int* __restrict__ chunk_count, const int* __restrict__ slots,
-                      const int* __restrict__ request_active, int heads, int cells, int max_slots, int* err) {
+                      const float* __restrict__ decays, const int* __restrict__ request_chunk_start,
+                      const int* __restrict__ slots, const int* __restrict__ request_active, int heads, int cells,
+                      int max_slots, int* err) {
   pdl_wait();
   pdl_trigger();
   const int request = blockIdx.x, head = blockIdx.y;
-  const int e = blockIdx.z * blockDim.x + threadIdx.x;
+  const int e = (blockIdx.z * blockDim.x + threadIdx.x) * V;
   if (e >= cells) return;
   const int slot = slots[request];
   if (slot < 0 || slot >= max_slots) {
@@ -281,28 +298,29 @@ ssd_chunk_walk_kernel(float* __restrict__ sums, float* __restrict__ state, long 
     return;
   }
   float* cell = state + (size_t)slot * state_stride + (size_t)head * cells + e;
-  float s = *cell;
+  float s[V];
+  load_v<V>(s, cell);
   const size_t stride = (size_t)heads * cells;
   const int last = request_chunk_start[request + 1];
   constexpr int kBatch = 8;          // the sums of eight chunks are asked for together, before the first store
   for (int chunk = request_chunk_start[request]; chunk < last; chunk += kBatch) {
     float* u = sums + ((size_t)chunk * heads + head) * cells + e;
-    float gained[kBatch], power[kBatch];
+    float gained[kBatch][V], keep[kBatch];
 #pragma unroll
     for (int b = 0; b < kBatch; ++b) {
-      const bool in = chunk + b < last;
-      gained[b] = in ? u[b * stride] : 0.f;
-      power[b] = in ? gates[(size_t)(chunk_row[chunk + b] + chunk_count[chunk + b] - 1) * heads + head].y : 0.f;
+      if (chunk + b >= last) break;
+      load_v<V>(gained[b], u + b * stride);
+      keep[b] = decays[(size_t)(chunk + b) * heads + head];
     }
 #pragma unroll
     for (int b = 0; b < kBatch; ++b) {
-      if (chunk + b < last) {
-        u[b * stride] = s;
-        s = fmaf(expf(power[b]), s, gained[b]);
-      }
+      if (chunk + b >= last) break;
+      store_v<V>(u + b * stride, s);
+#pragma unroll
+      for (int x = 0; x < V; ++x) s[x] = fmaf(keep[b], s[x], gained[b][x]);
     }
   }
-  if (request_active[request]) *cell = s;
+  if (request_active[request]) store_v<V>(cell, s);
 }
 
 // grid (chunks, heads, value tiles)
@@ -393,7 +411,8 @@ extern "C" int cie_ssd_scan(const float* rows, int stride, int x_off, int b_off,
 // Floats of scratch memory: gates, products, sums.
 extern "C" long long cie_ssd_chunk_floats(int tokens, int chunks, int heads, int groups, int n, int vdim) {
   const long long gates = ((long long)2 * tokens * heads + 3) / 4 * 4;
-  return gates + (long long)chunks * groups * kChunk * kChunk + (long long)chunks * heads * n * vdim;
+  const long long decays = ((long long)chunks * heads + 3) / 4 * 4;
+  return gates + decays + (long long)chunks * groups * kChunk * kChunk + (long long)chunks * heads * n * vdim;
 }
 
 extern "C" int cie_ssd_chunked(const float* rows, int stride, int x_off, int b_off, int c_off, const float* proj,
@@ -408,17 +427,24 @@ extern "C" int cie_ssd_chunked(const float* rows, int stride, int x_off, int b_o
   const Inputs in{rows, stride, x_off, b_off, c_off, proj, proj_stride, r_off, a_log, dt_bias, skip, heads, groups, n, vdim};
   cudaStream_t s = (cudaStream_t)stream;
   float2* gates = reinterpret_cast<float2*>(scratch);
-  float* products = scratch + ((long long)2 * tokens * heads + 3) / 4 * 4;
+  float* decays = scratch + ((long long)2 * tokens * heads + 3) / 4 * 4;
+  float* products = decays + ((long long)chunks * heads + 3) / 4 * 4;
   float* sums = products + (size_t)chunks * groups * kChunk * kChunk;
   const int state_tiles = (n + kTile - 1) / kTile, value_tiles = (vdim + kTile - 1) / kTile;
-  CIE_LAUNCH("ssd_gates", ssd_gates_kernel, dim3(chunks, (heads + 127) / 128), dim3(128), 0, s, in, gates, chunk_row, chunk_count);
+  CIE_LAUNCH("ssd_gates", ssd_gates_kernel, dim3(chunks, (heads + 127) / 128), dim3(128), 0, s, in, gates, decays, chunk_row, chunk_count);
   CIE_LAUNCH("ssd_chunk_products", ssd_chunk_products_kernel, dim3(chunks, groups), dim3(256), 0, s, in, products, chunk_row,
              chunk_count);
   CIE_LAUNCH("ssd_chunk_sums", ssd_chunk_sums_kernel, dim3(chunks, heads, state_tiles * value_tiles), dim3(256), 0, s, in,
              (const float2*)gates, sums, chunk_row, chunk_count);
-  CIE_LAUNCH("ssd_chunk_walk", ssd_chunk_walk_kernel, dim3(requests, heads, (n * vdim + 255) / 256), dim3(256), 0, s, sums,
-             state, state_stride, (const float2*)gates, request_chunk_start, chunk_row, chunk_count, slots, request_active,
-             heads, n * vdim, max_slots, err);
+  const int cells = n * vdim;
+  const bool wide = cells % 4 == 0 && state_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0;
+#define CIE_SSD_WALK(V)                                                                                              \
+  CIE_LAUNCH("ssd_chunk_walk", ssd_chunk_walk_kernel<V>, dim3(requests, heads, (cells + 128 * V - 1) / (128 * V)),   \
+             dim3(128), 0, s, sums, state, state_stride, (const float*)decays, request_chunk_start, slots,           \
+             request_active, heads, cells, max_slots, err)
+  if (wide) CIE_SSD_WALK(4);
+  else CIE_SSD_WALK(1);
+#undef CIE_SSD_WALK
   CIE_LAUNCH("ssd_chunk_output", ssd_chunk_output_kernel, dim3(chunks, heads, value_tiles), dim3(256), 0, s, in,
              (const float2*)gates, (const float*)products, (const float*)sums, out, out_stride, chunk_row, chunk_count);
   return 0;

@@ -21,6 +21,8 @@ NOISE = [None]      # a generator: what a 16-bit engine rounds (inputs of produc
 def rounded(x):
     if NOISE[0] is None:
         return x
+    if NOISE[0].initial_seed() == 0:
+        return x.to(torch.bfloat16).to(F64)
     return x * (1.0 + (torch.rand(x.shape, generator=NOISE[0], dtype=F64) - 0.5) * 2.0 ** -8)
 
 
@@ -245,7 +247,7 @@ def greedy(config, weights, prompt, count):
 def forward(config, weights, tokens, streams=None, noise=None):
     """Logits [T, vocab] of one sequence in float64.  ``streams``: a list that receives the stream after every
     layer.  ``noise``: a seed; inputs of products and rows that a cache holds are then each moved by up to the rounding
-    of bfloat16 (everything else stays exact)."""
+    of bfloat16, or (0) rounded to it; everything else stays exact."""
     NOISE[0] = None if noise is None else torch.Generator().manual_seed(noise)
     try:
         return _forward(config, weights, tokens, streams)
