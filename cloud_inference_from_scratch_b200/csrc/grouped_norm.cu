@@ -227,6 +227,135 @@ group_norm_kernel(float* residual, Update update, const float* __restrict__ gain
   });
 }
 
+// The same with the row in registers: P pieces of four elements a thread, every part on warps of its own; all loads of
+// a thread are asked for together.  Rows whose parts are whole pieces and fit.
+template <typename T, int P, int MODE>
+__global__ void __launch_bounds__(512)
+group_norm_pieces_kernel(float* residual, Update update, const float* __restrict__ gain, T* out, float* __restrict__ inv_out,
+                         const int* __restrict__ rows, Share share, float eps, Conv conv, int* err) {
+  __shared__ float scratch[33], warp_s[kMaxWarps];
+  const int hidden = share.part * share.groups;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = warp / share.wpg;
+  const int first = ((warp % share.wpg) * 32 + lane) * 4, step = share.wpg * 128;
+  const int column = g * share.part + first;
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.x, src = rows ? rows[r] : r;
+  float* res = residual + (size_t)src * hidden + column;
+  float x[P][4], w[P][4];
+#pragma unroll
+  for (int p = 0; p < P; ++p) {
+    const bool in = first + p * step < share.part;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[p][e] = w[p][e] = 0.f;
+    if (in) {
+      load_v<4>(x[p], res + p * step);
+      if (MODE == kNorm || MODE == kNormConv) load_v<4>(w[p], gain + column + p * step);
+    }
+  }
+  if (update.data != nullptr) {
+    const float* up = update.data + (size_t)src * hidden + column;
+    float y[P][4];
+#pragma unroll
+    for (int p = 0; p < P; ++p) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[p][e] = 0.f;
+      if (first + p * step < share.part) load_v<4>(y[p], up + p * step);
+    }
+    for (int s = 1; s < update.terms; ++s) {
+#pragma unroll
+      for (int p = 0; p < P; ++p) {
+        if (first + p * step >= share.part) continue;
+        float more[4];
+        load_v<4>(more, up + s * update.stride + p * step);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[p][e] += more[e];
+      }
+    }
+    if (update.gain == nullptr) {
+#pragma unroll
+      for (int p = 0; p < P; ++p)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[p][e] += y[p][e];
+    } else {
+      float gy[P][4], sq = 0.f;
+#pragma unroll
+      for (int p = 0; p < P; ++p) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) gy[p][e] = 0.f;
+        if (first + p * step < share.part) load_v<4>(gy[p], update.gain + column + p * step);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sq = fmaf(y[p][e], y[p][e], sq);
+      }
+      const float inv = rsqrtf(block_sum(sq, scratch) / (float)hidden + update.eps);
+#pragma unroll
+      for (int p = 0; p < P; ++p)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[p][e] = fmaf(y[p][e] * inv, gy[p][e], x[p][e]);
+    }
+    if (rows == nullptr)
+#pragma unroll
+      for (int p = 0; p < P; ++p)
+        if (first + p * step < share.part) store_v<4>(res + p * step, x[p]);
+  }
+  T* dst = out + (size_t)r * hidden + column;
+  if constexpr (MODE == kPlain) {
+#pragma unroll
+    for (int p = 0; p < P; ++p)
+      if (first + p * step < share.part) store_v<4>(dst + p * step, x[p]);
+    return;
+  }
+  float sq = 0.f;
+#pragma unroll
+  for (int p = 0; p < P; ++p)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) sq = fmaf(x[p][e], x[p][e], sq);
+  sq = warp_sum(sq);
+  if (share.wpg > 1) {
+    if (lane == 0) warp_s[warp] = sq;
+    __syncthreads();
+    sq = 0.f;
+    for (int k = 0; k < share.wpg; ++k) sq += warp_s[g * share.wpg + k];
+  }
+  const float inv = rsqrtf(sq / (float)share.part + eps);
+  if constexpr (MODE == kStats) {
+    if (lane == 0 && warp % share.wpg == 0) inv_out[(size_t)r * share.groups + g] = inv;
+    return;
+  }
+  float* hist = nullptr;
+  bool keep = false;
+  if constexpr (MODE == kNormConv) {
+    const int slot = conv.slots[r];
+    if (slot < 0 || slot >= conv.max_slots) {
+      if (threadIdx.x == 0) atomicOr(err, kErrBadRequest);
+      return;
+    }
+    hist = conv.history + (size_t)slot * conv.history_stride + column;
+    keep = conv.active[r] != 0;
+  }
+#pragma unroll
+  for (int p = 0; p < P; ++p) {
+    if (first + p * step >= share.part) continue;
+    float h[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) h[e] = w[p][e] * (x[p][e] * inv);
+    if constexpr (MODE == kNormConv) {
+      const float* f = conv.w + (size_t)(column + p * step) * conv.taps;
+      float acc[4] = {}, older[4];
+      for (int j = 0; j < conv.taps - 1; ++j) {
+        load_v<4>(older, hist + (size_t)j * hidden + p * step);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[e] = fmaf(f[e * conv.taps + j], older[e], acc[e]);
+        if (keep && j > 0) store_v<4>(hist + (size_t)(j - 1) * hidden + p * step, older);
+      }
+      if (keep && conv.taps > 1) store_v<4>(hist + (size_t)(conv.taps - 2) * hidden + p * step, h);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) h[e] += fmaf(f[e * conv.taps + conv.taps - 1], h[e], acc[e]);
+    }
+    store_v<4>(dst + p * step, h);
+  }
+}
+
 // h of token row t at channel i from the stream and the row's statistics.
 template <int V>
 __device__ __forceinline__ void normed(float (&h)[V], const float* __restrict__ stream, const float* __restrict__ inv,
@@ -400,6 +529,16 @@ static bool aligned16(const void* a, const void* b, const void* c, const void* d
            reinterpret_cast<uintptr_t>(d)) & 15) == 0;
 }
 
+// Pieces a thread of the kernel that keeps rows in registers would hold (0: not its kind).
+static int pieces_of(const Share& share, int threads) {
+  if (threads != 32 * share.wpg * share.groups || threads > 512) return 0;
+  const int pieces = (share.part + share.wpg * 128 - 1) / (share.wpg * 128);
+  return pieces <= 4 ? pieces : 0;
+}
+#define CIE_PIECES(name, P, MODE, count, out, inv, rows, conv, err)                                                  \
+  CIE_LAUNCH(name, (group_norm_pieces_kernel<T, P, MODE>), dim3(count), dim3(threads), 0, (cudaStream_t)stream,      \
+             residual, up, gain, (T*)(out), (float*)(inv), (const int*)(rows), share, eps, conv, (int*)(err))
+
 extern "C" int cie_norm_conv_max_taps() { return kMaxTaps; }
 
 // mode: 0 norm, 1 the rows themselves (gain unused).  out_dtype: float32 or bfloat16 (`out` may be the stream
@@ -418,6 +557,9 @@ extern "C" int cie_group_norm(float* residual, const float* update, int terms, l
   const bool wide = share.part % 4 == 0 && stride % 4 == 0 && aligned16(residual, update, gain, out) && aligned16(update_gain, 0, 0, 0);
 #define CIE_GROUP_NORM(V, MODE)                                                                                     \
   do {                                                                                                               \
+    if (V == 4 && pieces_of(share, threads) == 1) { CIE_PIECES("group_norm", 1, MODE, count, out, nullptr, rows, Conv{}, nullptr); break; } \
+    if (V == 4 && pieces_of(share, threads) == 2) { CIE_PIECES("group_norm", 2, MODE, count, out, nullptr, rows, Conv{}, nullptr); break; } \
+    if (V == 4 && pieces_of(share, threads) > 0) { CIE_PIECES("group_norm", 4, MODE, count, out, nullptr, rows, Conv{}, nullptr); break; } \
     if (allow_shared(group_norm_kernel<T, V, MODE>, smem, "group_norm")) return 1;                                   \
     CIE_LAUNCH("group_norm", (group_norm_kernel<T, V, MODE>), dim3(count), dim3(threads), smem, (cudaStream_t)stream, \
                residual, up, gain, (T*)out, (float*)nullptr, rows, share, eps, Conv{}, (int*)nullptr);               \
@@ -451,6 +593,13 @@ extern "C" int cie_group_norm_conv(float* residual, const float* update, int ter
                     aligned16(update_gain, history, 0, 0);
 #define CIE_CONV_STEP(V)                                                                                             \
   do {                                                                                                               \
+    const int pieces = V == 4 ? pieces_of(share, threads) : 0;                                                       \
+    if (singles && pieces) {                                                                                         \
+      if (pieces == 1) CIE_PIECES("group_norm_conv", 1, kNormConv, tokens, out, nullptr, nullptr, conv, err);        \
+      else if (pieces == 2) CIE_PIECES("group_norm_conv", 2, kNormConv, tokens, out, nullptr, nullptr, conv, err);   \
+      else CIE_PIECES("group_norm_conv", 4, kNormConv, tokens, out, nullptr, nullptr, conv, err);                    \
+      return 0;                                                                                                      \
+    }                                                                                                                \
     if (singles) {                                                                                                   \
       if (allow_shared(group_norm_kernel<T, V, kNormConv>, smem, "group_norm_conv")) return 1;                       \
       CIE_LAUNCH("group_norm_conv", (group_norm_kernel<T, V, kNormConv>), dim3(tokens), dim3(threads), smem,         \
@@ -458,9 +607,15 @@ extern "C" int cie_group_norm_conv(float* residual, const float* update, int ter
                  conv, err);                                                                                         \
       return 0;                                                                                                      \
     }                                                                                                                \
-    if (allow_shared(group_norm_kernel<T, V, kStats>, smem, "group_norm_conv")) return 1;                            \
-    CIE_LAUNCH("group_norm_stats", (group_norm_kernel<T, V, kStats>), dim3(tokens), dim3(threads), smem,             \
-               (cudaStream_t)stream, residual, up, gain, (T*)nullptr, inv, (const int*)nullptr, share, eps, conv, err); \
+    if (pieces == 1) CIE_PIECES("group_norm_stats", 1, kStats, tokens, nullptr, inv, nullptr, conv, err);            \
+    else if (pieces == 2) CIE_PIECES("group_norm_stats", 2, kStats, tokens, nullptr, inv, nullptr, conv, err);       \
+    else if (pieces) CIE_PIECES("group_norm_stats", 4, kStats, tokens, nullptr, inv, nullptr, conv, err);            \
+    else {                                                                                                           \
+      if (allow_shared(group_norm_kernel<T, V, kStats>, smem, "group_norm_conv")) return 1;                          \
+      CIE_LAUNCH("group_norm_stats", (group_norm_kernel<T, V, kStats>), dim3(tokens), dim3(threads), smem,           \
+                 (cudaStream_t)stream, residual, up, gain, (T*)nullptr, inv, (const int*)nullptr, share, eps, conv,  \
+                 err);                                                                                               \
+    }                                                                                                                \
     const int blocks = (hidden + V * kConvThreads - 1) / (V * kConvThreads);                                         \
     const dim3 grid((tokens + kConvRun - 1) / kConvRun, blocks);                                                     \
     if (taps == 2) CIE_CONV_RUN(V, 2); else if (taps == 3) CIE_CONV_RUN(V, 3);                                       \

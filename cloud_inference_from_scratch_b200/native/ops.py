@@ -699,7 +699,7 @@ class Ops:
                 "cie_ssd_scan", [v, i, i, i, i, v, i, i, v, v, v, v, i, v, ll, v, v, v, i, i, i, i, i, i, v, v])
             self._ssd_chunked = lib.function(
                 "cie_ssd_chunked",
-                [v, i, i, i, i, v, i, i, v, v, v, v, i, v, ll, v, v, v, v, v, v, i, i, i, i, i, i, i, i, v, v])
+                [v, i, i, i, i, v, i, i, v, v, v, v, i, v, ll, v, v, v, v, v, v, i, i, i, i, i, i, i, i, i, v, v])
             lib.handle.cie_ssd_chunk_floats.restype = ctypes.c_longlong
             self._ssd_chunk_floats = lib.handle.cie_ssd_chunk_floats
             self.ssd_max_state = int(lib.handle.cie_ssd_max_state())
@@ -743,10 +743,13 @@ class Ops:
             most = max(tokens, self.max_rows)
             reserve = int(self._ssd_chunk_floats(most, -(-most // self.ssd_chunk_tokens) + 64, heads, groups, dim, vdim))
             scratch = self.scratch(tag, floats, reserve=max(floats, reserve))
-            self.launches += 5
+            # 16-bit runs: the chunk products on the tensor cores, float32 operands as two bfloat16 terms each
+            tensor = self.code == BF16 and os.environ.get("CIE_SSD_TENSOR", "1") != "0"
+            self.launches += 4
             self._ssd_chunked(*head, _ptr(scratch), _ptr(plan["chunk_row"]), _ptr(plan["chunk_count"]),
                               _ptr(plan["request_chunk_start"]), _ptr(ctx.slots), _ptr(ctx.request_active), tokens, chunks,
-                              ctx.num_requests, heads, groups, dim, vdim, state.shape[0], _ptr(self.error_word), self.stream)
+                              ctx.num_requests, heads, groups, dim, vdim, state.shape[0], 1 if tensor else 0,
+                              _ptr(self.error_word), self.stream)
             return
         self.launches += 1
         self._ssd_scan(*head, _ptr(ctx.query_start), _ptr(ctx.slots), _ptr(ctx.request_active), ctx.num_requests, heads,
