@@ -177,7 +177,8 @@ __device__ __forceinline__ void stage_wait() {
 // kStaged: a warp first brings the key and value rows of its 32 keys into shared memory with
 // asynchronous 16-byte copies, all in flight at once (one trip to memory a block instead of one per
 // row piece), and reads them from there; rows of 16-bit elements whose sizes are multiples of 8.
-template <typename T, bool kStaged>
+// H: query heads a CTA works on (the smallest of 1, 2, 4 and 8 that holds its share of the group).
+template <typename T, bool kStaged, int H>
 __global__ void __launch_bounds__(kGroupWarps * 32)
 attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out, int out_stride,
                        const T* __restrict__ k_pool, const T* __restrict__ v_pool,
@@ -221,17 +222,17 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
     q_s[e] = h < heads ? to_float(q[(size_t)t * q_stride + (size_t)(kvh * group + h0 + h) * dim + d]) : 0.f;
   }
   const float *r1 = opt.r1, *sinks = opt.sinks;
-  float penalty[kGroupHeads], reach[kGroupHeads], slope[kGroupHeads];
+  float penalty[H], reach[H], slope[H];
 #pragma unroll
-  for (int h = 0; h < kGroupHeads; ++h) {
+  for (int h = 0; h < H; ++h) {
     penalty[h] = (r1 && h < heads) ? r1[kvh * group + h0 + h] : 0.f;
     reach[h] = (r1 && h < heads) ? opt.r2[kvh * group + h0 + h] : 0.f;
     slope[h] = (opt.slopes && h < heads) ? opt.slopes[kvh * group + h0 + h] : 0.f;
   }
   __syncthreads();
-  float m[kGroupHeads], l[kGroupHeads], acc[kGroupHeads][kGroupMaxV / 32];
+  float m[H], l[H], acc[H][kGroupMaxV / 32];
 #pragma unroll
-  for (int h = 0; h < kGroupHeads; ++h) {
+  for (int h = 0; h < H; ++h) {
     m[h] = -FLT_MAX;
     l[h] = 0.f;
 #pragma unroll
@@ -249,9 +250,9 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
       if (page < 0 || page >= num_pages) atomicOr(err, kErrBadPage);
       else slot = ((long long)page * kv_heads + kvh) * page_size + key % page_size;
     }
-    float dot[kGroupHeads];
+    float dot[H];
 #pragma unroll
-    for (int h = 0; h < kGroupHeads; ++h) dot[h] = 0.f;
+    for (int h = 0; h < H; ++h) dot[h] = 0.f;
     T* my_k = k_stage + ((size_t)warp * 32 + lane) * k_ld;
     T* my_v = v_stage + (size_t)warp * 32 * vdim;
     if constexpr (kStaged) {
@@ -271,13 +272,13 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
         for (int x = 0; x < V; ++x) {
           const float kf = to_float(kv[x]);
 #pragma unroll
-          for (int h = 0; h < kGroupHeads; ++h) dot[h] = fmaf(q_s[h * dim + d0 + x], kf, dot[h]);
+          for (int h = 0; h < H; ++h) dot[h] = fmaf(q_s[h * dim + d0 + x], kf, dot[h]);
         }
       }
     }
     const float distance = (float)(pos - key);
 #pragma unroll
-    for (int h = 0; h < kGroupHeads; ++h) {
+    for (int h = 0; h < H; ++h) {
       float s = -FLT_MAX;
       if (slot >= 0) {
         s = dot[h] * scale;
@@ -305,7 +306,7 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
 #pragma unroll
       for (int c = 0; c < kGroupMaxV / 32; ++c) vv[c] = lane + 32 * c < vdim ? to_float(vr[lane + 32 * c]) : 0.f;
 #pragma unroll
-      for (int h = 0; h < kGroupHeads; ++h) {
+      for (int h = 0; h < H; ++h) {
         const float pj = my_p[h * 32 + j];
 #pragma unroll
         for (int c = 0; c < kGroupMaxV / 32; ++c) acc[h][c] = fmaf(pj, vv[c], acc[h][c]);
@@ -315,7 +316,7 @@ attention_group_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
   }
   // ---- join the warps, in warp order
 #pragma unroll
-  for (int h = 0; h < kGroupHeads; ++h) {
+  for (int h = 0; h < H; ++h) {
 #pragma unroll
     for (int c = 0; c < kGroupMaxV / 32; ++c) o_s[(warp * kGroupHeads + h) * kGroupMaxV + lane + 32 * c] = acc[h][c];
     if (lane == 0) {
@@ -429,20 +430,28 @@ extern "C" int cie_attention_generic_sink(const void* q, int q_stride, void* out
     const bool staged = dtype == kBFloat16 && vdim % 8 == 0 && (reinterpret_cast<uintptr_t>(v_pool) & 15) == 0;
     const size_t smem = base + (staged ? (size_t)kGroupWarps * 32 * (dim + 8 + vdim) * sizeof(__nv_bfloat16) : 0);
     dim3 grid(tokens * splits, kv_heads, (group + kGroupHeads - 1) / kGroupHeads);
-#define CIE_GROUP(T, S)                                                                                            \
+#define CIE_GROUP_H(T, S, H)                                                                                           \
   do {                                                                                                             \
-    if (cudaFuncSetAttribute(attention_group_kernel<T, S>, cudaFuncAttributeMaxDynamicSharedMemorySize,            \
+    if (cudaFuncSetAttribute(attention_group_kernel<T, S, H>, cudaFuncAttributeMaxDynamicSharedMemorySize,            \
                              (int)smem) != cudaSuccess)                                                            \
       CIE_FAIL("attention_generic: cannot reserve %zu bytes of shared memory", smem);                              \
-    CIE_LAUNCH("attention_group", (attention_group_kernel<T, S>), grid, dim3(kGroupWarps * 32), smem, s,            \
+    CIE_LAUNCH("attention_group", (attention_group_kernel<T, S, H>), grid, dim3(kGroupWarps * 32), smem, s,            \
                (const T*)q, q_stride, (T*)out, out_stride, (const T*)k_pool, (const T*)v_pool, positions,          \
                request_of_token, table, table_width, num_pages, q_heads, kv_heads, dim, vdim, page_size, scale,    \
                window, keep_first, opt, splits, shares, tickets, err);                                   \
+  } while (0)
+#define CIE_GROUP(T, S)                              \
+  do {                                               \
+    if (group == 1) CIE_GROUP_H(T, S, 1);            \
+    else if (group == 2) CIE_GROUP_H(T, S, 2);       \
+    else if (group <= 4) CIE_GROUP_H(T, S, 4);       \
+    else CIE_GROUP_H(T, S, 8);                       \
   } while (0)
     if (dtype == kFloat32) CIE_GROUP(float, false);
     else if (staged) CIE_GROUP(__nv_bfloat16, true);
     else CIE_GROUP(__nv_bfloat16, false);
 #undef CIE_GROUP
+#undef CIE_GROUP_H
     return 0;
   }
   if (dtype == kFloat32) {

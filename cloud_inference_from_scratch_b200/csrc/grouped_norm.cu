@@ -2,7 +2,8 @@
 // and what sits right beside them in a layer:
 //
 //  * group_norm        the pending update joins the float32 stream, then the norm: out = gain * (x / rms of its part).
-//                      The update is a sum of float32 terms, or such a sum that is itself RMS-normalised over the
+//                      The update is a sum of float32 terms (plain, or weighted by a number per row and term: a
+//                      token's expert outputs), or such a sum that is itself RMS-normalised over the
 //                      whole row and multiplied by a gain vector before it is added (`update_gain`).
 //  * stream_rows       the same add, and the stream's own rows rounded to the activation type (no norm)
 //  * group_norm_conv   the same norm followed by a causal convolution over time on every channel whose result is
@@ -22,7 +23,7 @@ CIE_DEFINE_LAST_ERROR()
 namespace cie {
 
 constexpr int kMaxTaps = 16;     // longest convolution
-constexpr int kMaxTerms = 8;     // float32 terms of a pending update
+constexpr int kMaxTerms = 32;    // float32 terms of a pending update
 constexpr int kMaxWarps = 32;
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
@@ -90,19 +91,20 @@ __device__ __forceinline__ void part_inverses(const Share& share, const float* u
 }
 
 struct Update {
-  const float* data;      // float32 terms [terms][rows][hidden], `stride` apart; nullptr: nothing pending
+  const float* data;      // float32 terms: term s of row r at r * row_stride + s * stride; nullptr: nothing pending
   int terms;
-  size_t stride;
+  size_t stride, row_stride;
+  const float* weights;   // not null: term s of row r is multiplied by weights[r * terms + s]
   const float* gain;      // not null: the sum is RMS-normalised over the whole row and multiplied by this first
   float eps;
 };
 
 // The row of the stream with its update applied, in u_s (and in the stream, unless write_back is false).
 template <int V>
-__device__ __forceinline__ void stream_row(const Share& share, float* residual, const Update& update, size_t offset,
+__device__ __forceinline__ void stream_row(const Share& share, float* residual, const Update& update, int row,
                                            bool write_back, float* u_s, float* scratch) {
   const int hidden = share.part * share.groups;
-  float* res = residual + offset;
+  float* res = residual + (size_t)row * hidden;
   if (update.data == nullptr) {
     share.each<V>([&](int, int i) {
       float x[V];
@@ -111,14 +113,19 @@ __device__ __forceinline__ void stream_row(const Share& share, float* residual, 
     });
     return;
   }
-  const float* up = update.data + offset;
+  const float* up = update.data + (size_t)row * update.row_stride;
+  const float* weights = update.weights ? update.weights + (size_t)row * update.terms : nullptr;
   auto pending = [&](int i, float (&y)[V]) {
     load_v<V>(y, up + i);
+    if (weights)
+#pragma unroll
+      for (int x = 0; x < V; ++x) y[x] *= weights[0];
     for (int s = 1; s < update.terms; ++s) {
       float more[V];
       load_v<V>(more, up + s * update.stride + i);
+      const float w = weights ? weights[s] : 1.f;
 #pragma unroll
-      for (int x = 0; x < V; ++x) y[x] += more[x];
+      for (int x = 0; x < V; ++x) y[x] = fmaf(w, more[x], y[x]);
     }
   };
   if (update.gain == nullptr) {
@@ -179,7 +186,7 @@ group_norm_kernel(float* residual, Update update, const float* __restrict__ gain
   pdl_wait();
   pdl_trigger();
   const int r = blockIdx.x, src = rows ? rows[r] : r;
-  stream_row<V>(share, residual, update, (size_t)src * hidden, rows == nullptr, u_s, scratch);
+  stream_row<V>(share, residual, update, src, rows == nullptr, u_s, scratch);
   T* dst = out + (size_t)r * hidden;
   if constexpr (MODE == kPlain) {
     share.each<V>([&](int, int i) {
@@ -254,22 +261,28 @@ group_norm_pieces_kernel(float* residual, Update update, const float* __restrict
     }
   }
   if (update.data != nullptr) {
-    const float* up = update.data + (size_t)src * hidden + column;
+    const float* up = update.data + (size_t)src * update.row_stride + column;
+    const float* weights = update.weights ? update.weights + (size_t)src * update.terms : nullptr;
+    const float w0 = weights ? weights[0] : 1.f;
     float y[P][4];
 #pragma unroll
     for (int p = 0; p < P; ++p) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) y[p][e] = 0.f;
       if (first + p * step < share.part) load_v<4>(y[p], up + p * step);
+      if (weights)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[p][e] *= w0;
     }
     for (int s = 1; s < update.terms; ++s) {
+      const float ws = weights ? weights[s] : 1.f;
 #pragma unroll
       for (int p = 0; p < P; ++p) {
         if (first + p * step >= share.part) continue;
         float more[4];
         load_v<4>(more, up + s * update.stride + p * step);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) y[p][e] += more[e];
+        for (int e = 0; e < 4; ++e) y[p][e] = fmaf(ws, more[e], y[p][e]);
       }
     }
     if (update.gain == nullptr) {
@@ -387,6 +400,8 @@ norm_conv_kernel(const float* __restrict__ stream, const float* __restrict__ inv
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) w[e][j] = conv.w[(size_t)(i + e) * TAPS + j];
   const int t0 = blockIdx.x * kConvRun, t1 = min(t0 + kConvRun, tokens);
+  float window[TAPS ? TAPS : 1][V];      // h of the request's last TAPS tokens
+  int held = -1;                         // the request they belong to
   for (int t = t0; t < t1; ++t) {
     const int request = request_of_token[t], begin = query_start[request];
     const int slot = conv.slots[request];
@@ -395,25 +410,37 @@ norm_conv_kernel(const float* __restrict__ stream, const float* __restrict__ inv
       return;
     }
     const float* hist = conv.history + (size_t)slot * conv.history_stride;
-    float acc[V] = {}, h[V];
-    auto tap = [&](int j) {
-      const int src = t - begin - (taps - 1 - j);
+    auto fetch = [&](float (&h)[V], int src) {       // h of the request's token `src` of this step (< 0: an earlier one)
       if (src >= 0) normed<V>(h, stream, inv, gv, begin + src, i, g, hidden, groups);
       else load_v<V>(h, hist + (size_t)(taps - 1 + src) * hidden + i);
-#pragma unroll
-      for (int e = 0; e < V; ++e) {
-        if constexpr (TAPS > 0) acc[e] = fmaf(w[e][j], h[e], acc[e]);
-        else acc[e] = fmaf(conv.w[(size_t)(i + e) * taps + j], h[e], acc[e]);
-      }
     };
+    float acc[V] = {}, h[V];
     if constexpr (TAPS > 0) {
+      if (request != held) {             // the run's first token, or another request's: fill the window
+        held = request;
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) tap(j);
+        for (int j = 1; j < TAPS; ++j) fetch(window[j], t - begin - (TAPS - j));
+      }
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < V; ++e) window[j][e] = window[j + 1][e];
+      fetch(window[TAPS - 1], t - begin);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e][j], window[j][e], acc[e]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) h[e] = window[TAPS - 1][e] + acc[e];
     } else {
-      for (int j = 0; j < taps; ++j) tap(j);
-    }
+      for (int j = 0; j < taps; ++j) {
+        fetch(h, t - begin - (taps - 1 - j));
 #pragma unroll
-    for (int e = 0; e < V; ++e) h[e] += acc[e];       // the last tap read the token's own row
+        for (int e = 0; e < V; ++e) acc[e] = fmaf(conv.w[(size_t)(i + e) * taps + j], h[e], acc[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) h[e] += acc[e];       // the last tap read the token's own row
+    }
     store_v<V>(out + (size_t)t * hidden + i, h);
   }
 }
@@ -543,8 +570,8 @@ extern "C" int cie_norm_conv_max_taps() { return kMaxTaps; }
 
 // mode: 0 norm, 1 the rows themselves (gain unused).  out_dtype: float32 or bfloat16 (`out` may be the stream
 // itself in float32: a row is read whole before it is written).
-extern "C" int cie_group_norm(float* residual, const float* update, int terms, long long stride, const float* update_gain,
-                              float update_eps, const float* gain, void* out, const int* rows, int count, int hidden,
+extern "C" int cie_group_norm(float* residual, const float* update, int terms, long long stride, long long row_stride,
+                              const float* weights, const float* update_gain, float update_eps, const float* gain, void* out, const int* rows, int count, int hidden,
                               int groups, float eps, int mode, int out_dtype, void* stream) {
   if (count <= 0) return 0;
   if (groups < 1 || hidden < 1 || hidden % groups) CIE_FAIL("group_norm: a row of %d in %d parts", hidden, groups);
@@ -552,9 +579,9 @@ extern "C" int cie_group_norm(float* residual, const float* update, int terms, l
   if (mode != kNorm && mode != kPlain) CIE_FAIL("group_norm: unknown mode %d", mode);
   Share share;
   const int threads = share_row(&share, hidden, groups);
-  const Update up{update, terms, (size_t)stride, update_gain, update_eps};
+  const Update up{update, terms, (size_t)stride, (size_t)row_stride, weights, update_gain, update_eps};
   const size_t smem = (size_t)(((hidden + 3) & ~3) + groups) * sizeof(float);
-  const bool wide = share.part % 4 == 0 && stride % 4 == 0 && aligned16(residual, update, gain, out) && aligned16(update_gain, 0, 0, 0);
+  const bool wide = share.part % 4 == 0 && stride % 4 == 0 && row_stride % 4 == 0 && aligned16(residual, update, gain, out) && aligned16(update_gain, 0, 0, 0);
 #define CIE_GROUP_NORM(V, MODE)                                                                                     \
   do {                                                                                                               \
     if (V == 4 && pieces_of(share, threads) == 1) { CIE_PIECES("group_norm", 1, MODE, count, out, nullptr, rows, Conv{}, nullptr); break; } \
@@ -573,8 +600,8 @@ extern "C" int cie_group_norm(float* residual, const float* update, int terms, l
 }
 
 // singles: every request brings one token (row t is request t).  inv: float32 scratch [tokens][groups], used otherwise.
-extern "C" int cie_group_norm_conv(float* residual, const float* update, int terms, long long stride,
-                                   const float* update_gain, float update_eps, const float* gain, void* out, float* inv,
+extern "C" int cie_group_norm_conv(float* residual, const float* update, int terms, long long stride, long long row_stride,
+                                   const float* weights, const float* update_gain, float update_eps, const float* gain, void* out, float* inv,
                                    const float* w, int taps, float* history, long long history_stride,
                                    const int* query_start, const int* request_of_token, const int* slots,
                                    const int* request_active, int tokens, int requests, int max_slots, int hidden,
@@ -586,10 +613,10 @@ extern "C" int cie_group_norm_conv(float* residual, const float* update, int ter
   if (singles && tokens != requests) CIE_FAIL("group_norm_conv: %d tokens of %d requests are not single tokens", tokens, requests);
   Share share;
   const int threads = share_row(&share, hidden, groups);
-  const Update up{update, terms, (size_t)stride, update_gain, update_eps};
+  const Update up{update, terms, (size_t)stride, (size_t)row_stride, weights, update_gain, update_eps};
   const Conv conv{w, taps, history, history_stride, slots, request_active, max_slots};
   const size_t smem = (size_t)(((hidden + 3) & ~3) + groups) * sizeof(float);
-  const bool wide = share.part % 4 == 0 && stride % 4 == 0 && history_stride % 4 == 0 && aligned16(residual, update, gain, out) &&
+  const bool wide = share.part % 4 == 0 && stride % 4 == 0 && row_stride % 4 == 0 && history_stride % 4 == 0 && aligned16(residual, update, gain, out) &&
                     aligned16(update_gain, history, 0, 0);
 #define CIE_CONV_STEP(V)                                                                                             \
   do {                                                                                                               \

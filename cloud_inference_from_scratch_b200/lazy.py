@@ -110,6 +110,19 @@ class NormedUpdate:
         return tuple(self.y.shape)
 
 
+class WeightedTerms:
+    """A weighted sum that has not been taken yet: row t is ``sum_j weights[t, j] * terms[t, j]``, with ``terms`` float32
+    [T, count * H] (the ``count`` terms of a row side by side) and ``weights`` float32 [T, count].  The norm that reads the
+    stream next takes it in its own kernel, in float32, in ascending order."""
+
+    def __init__(self, terms: Any, weights: Any) -> None:
+        self.terms, self.weights, self.count = terms, weights, int(weights.shape[1])
+
+    @property
+    def shape(self) -> tuple[int, ...]:
+        return (int(self.terms.shape[0]), int(self.terms.shape[1]) // self.count)
+
+
 class PendingNorm:
     """A norm that has not run yet, with what it needs: the stream, the update that still has to join it, gain, eps and
     the number of parts.  Whoever takes this instead of a tensor (``takes_pending_norm``) runs the norm as the first

@@ -68,7 +68,7 @@ def sutuvik_spec(config: SutuvikConfig) -> ModelSpec:
                 "routed_experts", dict(hidden_size=config.width, intermediate_size=layer.mlp.ff,
                                        num_experts=layer.mlp.experts, top=layer.mlp.top, correction=True,
                                        renormalize=True, score="sigmoid", groups=(layer.mlp.groups, layer.mlp.keep),
-                                       norm_floor=WEIGHT_FLOOR), prefix="mlp.")
+                                       norm_floor=WEIGHT_FLOOR, defer_sum=True), prefix="mlp.")
         layers.append(LayerSpec(prefix=f"l{index}.", block=PartSpec("prenorm_residual"), parts=parts))
     return ModelSpec(
         architecture=config.architecture,

@@ -15,7 +15,7 @@ import os
 from ctypes import c_float, c_int, c_void_p
 from typing import Any
 
-from ..lazy import Accumulated, GateUpWeight, NormedInput, NormedUpdate, Partials, ResidualSink, StreamUpdate  # noqa: F401  (re-exported)
+from ..lazy import Accumulated, GateUpWeight, NormedInput, NormedUpdate, Partials, ResidualSink, StreamUpdate, WeightedTerms  # noqa: F401  (re-exported)
 from .build import load_library
 
 F32, BF16 = 0, 1
@@ -237,6 +237,12 @@ class Ops:
 
     def require_attention(self, head_dim: int) -> None:
         """Builds, at model set-up, the attention kernels a head size needs."""
+        self.require_portion_attention(head_dim)
+        if head_dim in self._tensor_attention:
+            self._tensor_attention[head_dim].load_prompt_kernel()
+
+    def require_portion_attention(self, head_dim: int) -> None:
+        """The same for a layer with options of ``attention_penalised``, which the tcgen05 prompt kernel does not take."""
         if self.code == BF16:
             from . import tensor_attention
 
@@ -606,10 +612,10 @@ class Ops:
         if self._grouped_lib is None:
             v, i, f, ll = c_void_p, c_int, c_float, ctypes.c_longlong
             lib = _Lib(load_library("grouped_norm.cu"))
-            self._group_norm = lib.function("cie_group_norm", [v, v, i, ll, v, f, v, v, v, i, i, i, f, i, i, v])
+            self._group_norm = lib.function("cie_group_norm", [v, v, i, ll, ll, v, v, f, v, v, v, i, i, i, f, i, i, v])
             self._group_norm_conv = lib.function(
                 "cie_group_norm_conv",
-                [v, v, i, ll, v, f, v, v, v, v, i, v, ll, v, v, v, v, i, i, i, i, i, f, i, i, v, v])
+                [v, v, i, ll, ll, v, v, f, v, v, v, v, i, v, ll, v, v, v, v, i, i, i, i, i, f, i, i, v, v])
             self._gated_group_norm = lib.function("cie_gated_group_norm", [v, i, v, i, v, v, i, i, i, i, f, i, v])
             self._side_gate = lib.function("cie_side_gate", [v, v, v, i, i, i, v, i, i, i, v, v])
             self.norm_conv_max_taps = int(lib.handle.cie_norm_conv_max_taps())
@@ -620,9 +626,10 @@ class Ops:
         self._load_grouped()
         return self.norm_conv_max_taps
 
-    def _pending_terms(self, update: Any) -> tuple[Any, int, int, Any, float]:
-        """A pending update as float32 terms: (tensor or None, terms, stride, gain or None, eps)."""
-        gain, eps = None, 0.0
+    def _pending_terms(self, update: Any, hidden: int) -> tuple[Any, ...]:
+        """A pending update as the kernels take it: pointer or None, terms, strides from term to term and row to row,
+        weights, gain, eps (and what must stay alive until the launch)."""
+        gain, eps, weights = None, 0.0, None
         if isinstance(update, NormedUpdate):
             gain, eps, update = update.gain, update.eps, update.y
         if isinstance(update, Accumulated):
@@ -630,23 +637,26 @@ class Ops:
         if isinstance(update, Partials) and (update.splits == 0 or update.bias is not None):
             update = self.resolve(update, self.torch.empty(update.shape, dtype=self.torch.float32, device=self.device))
         if update is None:
-            return None, 0, 0, None, 0.0
-        if isinstance(update, Partials):
-            return update.data, update.splits, update.stride, gain, eps
-        return (update if update.dtype == self.torch.float32 else update.float()), 1, 0, gain, eps
+            return (None, 0, 0, 0, None, None, 0.0), None
+        if isinstance(update, WeightedTerms):
+            data, terms, stride, row_stride, weights = update.terms, update.count, hidden, update.count * hidden, update.weights
+        elif isinstance(update, Partials):
+            data, terms, stride, row_stride = update.data, update.splits, update.stride, hidden
+        else:
+            data, terms, stride, row_stride = update if update.dtype == self.torch.float32 else update.float(), 1, 0, hidden
+        return (_ptr(data), terms, stride, row_stride, _ptr(weights), _ptr(gain), float(eps)), data
 
     def group_norm(self, residual: Any, update: Any, gain: Any, eps: float, groups: int, out: Any, rows: Any = None) -> None:
         """The pending update joins the float32 stream, and ``out`` is the norm of its rows in ``groups`` equal
         consecutive parts, each divided by its own root mean square, times ``gain``; ``gain`` None: the rows
-        themselves, rounded.  ``update``: None, a tensor, ``Partials`` or a ``NormedUpdate``.  With ``rows`` only those
+        themselves, rounded.  ``update``: None, a tensor, ``Partials``, ``WeightedTerms`` or a ``NormedUpdate``.  With ``rows`` only those
         rows are read and the stream stays as it was.  ``out`` may be the stream itself."""
         self._flush()
         self._load_grouped()
         count, hidden = out.shape
-        data, terms, stride, update_gain, update_eps = self._pending_terms(update)
+        pending, held = self._pending_terms(update, hidden)
         self.launches += 1
-        self._group_norm(_ptr(residual), _ptr(data), terms, stride, _ptr(update_gain), float(update_eps), _ptr(gain),
-                         _ptr(out), _ptr(rows), count, hidden, groups, float(eps), 1 if gain is None else 0,
+        self._group_norm(_ptr(residual), *pending, _ptr(gain), _ptr(out), _ptr(rows), count, hidden, groups, float(eps), 1 if gain is None else 0,
                          self._code_of(out), self.stream)
 
     def group_norm_conv(self, residual: Any, update: Any, gain: Any, eps: float, groups: int, weight: Any, history: Any,
@@ -658,15 +668,14 @@ class Ops:
         self._load_grouped()
         tokens, hidden = out.shape
         taps = weight.shape[1]
-        data, terms, stride, update_gain, update_eps = self._pending_terms(update)
+        pending, held = self._pending_terms(update, hidden)
         singles = tokens == ctx.num_requests and ctx.num_single == ctx.num_requests
         inverses = None
         if not singles:
             inverses = self.scratch(f"norm_conv.inverses.{groups}", tokens * groups,
                                     reserve=max(tokens, self.max_rows) * groups)
         self.launches += 1 if singles else (3 if taps > 1 else 2)
-        self._group_norm_conv(_ptr(residual), _ptr(data), terms, stride, _ptr(update_gain), float(update_eps), _ptr(gain),
-                              _ptr(out), _ptr(inverses), _ptr(weight), taps, _ptr(history),
+        self._group_norm_conv(_ptr(residual), *pending, _ptr(gain), _ptr(out), _ptr(inverses), _ptr(weight), taps, _ptr(history),
                               history.stride(0) if history is not None else 0, _ptr(ctx.query_start),
                               _ptr(ctx.request_of_token), _ptr(ctx.slots), _ptr(ctx.request_active), tokens,
                               ctx.num_requests, history.shape[0] if history is not None else 1 << 30, hidden, groups,
@@ -1229,7 +1238,7 @@ class Ops:
     def routed_experts(self, x: Any, router: Any, correction: Any, w_gate: Any, w_up: Any, w_down: Any,
                        top: int, renormalize: bool, out: Any, workspace: Any, router_bias: Any = None,
                        chosen_softmax: bool = False, sigmoid: bool = False, groups: tuple[int, int] = (1, 1),
-                       norm_floor: float = 0.0) -> Any:
+                       norm_floor: float = 0.0, defer: bool = False) -> Any:
         """out[t] = sum over the ``top`` chosen experts e of score_e * down_e(SiLU(gate_e x) * up_e x).
         ``router`` float32 [E, H]; ``w_gate``/``w_up`` [E, F, H], or ``w_up`` None and ``w_gate`` the
         interleaved [E, 2F, H] of ``interleave_gate_up``; ``w_down`` [E, H, F]; ``out`` float32 or the
@@ -1237,7 +1246,8 @@ class Ops:
         experts with the largest logits are chosen and weighted by the softmax over their logits alone;
         ``sigmoid``: scores are sigmoids of the logits; ``groups`` = (count, keep): experts form equal groups of
         neighbours and only those of the ``keep`` groups whose two largest choice scores have the largest sums can
-        be chosen; ``norm_floor`` is added to the sum that ``renormalize`` divides by."""
+        be chosen; ``norm_floor`` is added to the sum that ``renormalize`` divides by.  ``defer``: the weighted sum is
+        left to the kernel that reads the stream next (``out`` is not written; ``WeightedTerms`` is returned)."""
         self._flush()
         self._load_moe()
         torch = self.torch
@@ -1289,6 +1299,9 @@ class Ops:
                                    _ptr(tile_count), tokens, top, experts, ff, hidden, code, self.stream)
             self._moe_down_simt(_ptr(act), _ptr(w_down), _ptr(rows), _ptr(place_to_pair), _ptr(tiles),
                                 _ptr(tile_count), tokens, top, experts, ff, hidden, code, self.stream)
+        if defer:
+            self.launches -= 1
+            return WeightedTerms(rows, weights)
         self._moe_combine(_ptr(rows), _ptr(weights), _ptr(out), tokens, hidden, top, self._code_of(out), self.stream)
         return out
 

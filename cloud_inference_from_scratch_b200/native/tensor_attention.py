@@ -138,10 +138,16 @@ class TensorAttention:
             self._split_tickets = ops.torch.zeros(self.split_cta_limit, dtype=ops.torch.int32, device=ops.device)
 
         self.use_tma = 0 if os.environ.get("CIE_DECODE_TMA", "1") == "0" else 1
-        # prompt portions on tcgen05 where the kernel exists: head size 64 or 128, no window,
-        # pages of a multiple of 16 tokens; everything else stays on the mma.sync kernel
         self._prefill_tc = None
-        if head_dim in (64, 128) and os.environ.get("CIE_PREFILL_TC", "1") != "0":
+
+    def load_prompt_kernel(self) -> None:
+        """Prompt portions on tcgen05 where the kernel exists: head size 64 or 128, no window, pages of a multiple
+        of 16 tokens; everything else stays on the mma.sync kernel (``run_portions`` alone never needs this one)."""
+        from .ops import _Lib
+
+        head_dim, torch, ops = self.head_dim, self.ops.torch, self.ops
+        v, i, f = c_void_p, c_int, c_float
+        if self._prefill_tc is None and head_dim in (64, 128) and os.environ.get("CIE_PREFILL_TC", "1") != "0":
             defines = {"HEAD_DIM": head_dim}
             for name in ("TC_BN", "TC_STAGES", "TC_KEY_PRODUCERS", "TC_VALUE_PRODUCERS"):
                 if os.environ.get("CIE_" + name):

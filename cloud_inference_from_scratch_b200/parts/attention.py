@@ -259,8 +259,10 @@ class Attention(Mixer):
         # the tensor-core kernels take bfloat16 heads of a multiple of 16 elements, keys and values alike or not
         self.tiled = bool(self.value_dim % 16 == 0 and self.head_dim % 16 == 0 and max(self.head_dim, self.value_dim) <= 256
                           and runtime.dtype_name == "bfloat16")
-        if not self.general or self.tiled:
-            runtime.ops.require_attention(max(self.head_dim, self.value_dim))
+        if not self.general:
+            runtime.ops.require_attention(self.head_dim)
+        elif self.tiled:
+            runtime.ops.require_portion_attention(max(self.head_dim, self.value_dim))
 
     takes_normed_input = True   # x goes to ops.linear only
     kernels_through_ops = True  # every kernel of this part is a method of ``Ops``: a decode step may be recorded

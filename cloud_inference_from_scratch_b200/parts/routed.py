@@ -15,7 +15,8 @@ experts with the largest logits and weights them by the softmax over the chosen 
 
 ``score="sigmoid"`` makes the scores sigmoids of the logits.  ``groups`` = (count, keep): the experts form ``count``
 equal groups of neighbours, a group's score is the sum of its two largest choice scores (score + correction), and only
-experts of the ``keep`` best groups can be chosen.  ``norm_floor`` is added to the sum that ``renormalize`` divides by.
+experts of the ``keep`` best groups can be chosen.  ``norm_floor`` is added to the sum that ``renormalize`` divides by.  ``defer_sum``: the weighted sum over the chosen
+experts is left to whoever reads the stream next (``WeightedTerms``; for norms that take it).
 
 The kernels group the (token, expert) pairs by expert on the device and never tell the host how
 many tokens an expert got, so a step is one fixed sequence of launches.
@@ -30,7 +31,7 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, intermediate_size: int, num_experts: int, top: int,
                  correction: bool = True, renormalize: bool = False,
                  names: dict[str, str] | None = None, router_bias: bool = False, score: str = "softmax",
-                 groups: tuple[int, int] = (1, 1), norm_floor: float = 0.0) -> None:
+                 groups: tuple[int, int] = (1, 1), norm_floor: float = 0.0, defer_sum: bool = False) -> None:
         if not 1 <= top <= num_experts:
             raise ValueError("top must lie in 1..num_experts")
         self.hidden_size = int(hidden_size)
@@ -49,6 +50,7 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed experts: groups are built for a choice among scores, not among logits")
         self.groups = (count, keep)
         self.norm_floor = float(norm_floor)
+        self.defer_sum = bool(defer_sum)
         if score == "chosen_softmax" and correction:
             raise ValueError("routed experts: a correction steers a choice among softmax scores, not among logits")
         self.score = score
@@ -94,7 +96,8 @@ class RoutedExperts(FeedForward):
         return rt.ops.routed_experts(x, self.router, self.bias, self.w_gate, self.w_up, self.w_down,
                                      self.top, self.renormalize, update, rt.workspace, router_bias=self.logit_bias,
                                      chosen_softmax=self.score == "chosen_softmax",
-                                     sigmoid=self.score == "sigmoid", groups=self.groups, norm_floor=self.norm_floor)
+                                     sigmoid=self.score == "sigmoid", groups=self.groups, norm_floor=self.norm_floor,
+                                     defer=self.defer_sum)
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts, replace=True)

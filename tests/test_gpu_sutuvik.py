@@ -321,14 +321,16 @@ def plan_into(ctx, rt, group):
 
 def updates_for(rows, width, rt):
     """Every kind of pending update with the plain value that joins the stream."""
-    from cloud_inference_from_scratch_b200.lazy import NormedUpdate, Partials
+    from cloud_inference_from_scratch_b200.lazy import NormedUpdate, Partials, WeightedTerms
 
     first, second = rand(rows, width, seed=4), rand(rows, width, seed=5)
     both = torch.stack([first, second]).cuda().contiguous()
-    gain = 1 + rand(width, scale=0.3, seed=6)
+    gain, share = 1 + rand(width, scale=0.3, seed=6), rand(rows, 3, seed=7)
     return [(None, torch.zeros(rows, width, dtype=F)), (first.cuda(), first.double()),
             (Partials(both, 2, rows, width, None), (first + second).double()),
             (first.to(rt.dtype).cuda(), first.to(rt.dtype).double()),
+            (WeightedTerms(torch.cat([first, second, first * second], 1).cuda(), share.cuda()),
+             (torch.stack([first, second, first * second], 1).double() * share.double().unsqueeze(-1)).sum(1)),
             (NormedUpdate(first.cuda(), gain.cuda(), 1e-5), plain.rms(first.double(), 1e-5) * gain.double())]
 
 
@@ -439,7 +441,7 @@ def test_biased_attention_far_keys_edges_and_a_sink(dtype, dim, vdim, group):
     groups, page, eps, n = 2, 16, 1e-5, 300
     heads = groups * group
     scale, coef, every = 6.0 / dim ** 0.5, 0.3, 64
-    rt.ops.require_attention(max(dim, vdim))
+    rt.ops.require_portion_attention(max(dim, vdim))
     width = heads * dim + groups * (dim + vdim)
     q_gain, k_gain = 1 + rand(dim, scale=0.2, seed=3), 1 + rand(dim, scale=0.2, seed=4)
     sink, slopes, gates = rand(heads, scale=3.0, seed=5), plain.head_slopes(heads), rand(n, heads + 3, scale=2.0, seed=6)
@@ -482,7 +484,7 @@ def test_rotated_attention_unit_size_factor_cap_and_one_in_the_denominator(dtype
     heads = groups * group
     scale = 2.0 * cap / dim
     rot = dict(base=2000.0, dims=dims, scaling=dict(factor=6.0, low=1.0, high=4.0, original=128))
-    rt.ops.require_attention(max(dim, vdim))
+    rt.ops.require_portion_attention(max(dim, vdim))
     width = heads * dim + groups * (dim + vdim)
     factor = 1 + rand(heads, scale=0.4, seed=7)
     for edge in (0, 37, page * 9 - 1, page * 9, n - 1):
