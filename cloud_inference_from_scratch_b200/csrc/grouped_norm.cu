@@ -27,8 +27,10 @@ constexpr int kMaxTerms = 32;    // float32 terms of a pending update
 constexpr int kMaxWarps = 32;
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// 0.5 z (1 + tanh(u)) with u = sqrt(2 / pi) (z + 0.044715 z^3), as z sigmoid(2 u): the same function without the
+// cancellation of 1 + tanh for negative z, which a norm of the results would blow up.
 __device__ __forceinline__ float gelu_tanh_f(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
+  return z / (1.f + expf(-2.f * 0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
 }
 
 template <int V> __device__ __forceinline__ void load_v(float (&dst)[V], const float* src) {
