@@ -145,7 +145,7 @@ class CachePools:
         self.pages_per_group = list(pages_per_group)
         self.states: dict[int, Any] = {}
         for need in needs:
-            if need.state is not None and need.owner == need.entry:
+            if need.state is not None and need.state_owner == need.entry:
                 self.states[need.entry] = torch.zeros(
                     (max_slots, *need.state.shape), dtype=getattr(torch, need.state.dtype),
                     device=device,
@@ -161,7 +161,7 @@ class CachePools:
                                  num_pages=pages_per_group[group], page_size=page_size)
             self.bindings.append(
                 LayerBinding(entry=need.entry, owns_cache=need.owner == need.entry, kv=kv,
-                             state=self.states.get(need.owner))
+                             state=self.states.get(need.state_owner))
             )
 
     def zero_slots(self, slots: list[int]) -> None:

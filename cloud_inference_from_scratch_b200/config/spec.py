@@ -87,6 +87,8 @@ class ScheduleEntry:
     ``reads_cache_of``  index of an EARLIER schedule entry whose cache (pages and
                    per-request state) this run reads instead of owning one; then it
                    writes nothing to a cache.
+    ``own_state``  with ``reads_cache_of``: only the pages are the other run's; the per-request
+                   state is this run's own.
     ``entry_offset``  (tensor name, row): row ``row`` of the stored tensor [rows, hidden] is
                    added to the residual stream of every token right before this run (a
                    learned offset per pass of a looped run of layers).
@@ -98,6 +100,7 @@ class ScheduleEntry:
     reads_cache_of: int | None = None
     entry_offset: tuple[str, int] | None = None
     adds_embedding: bool = False
+    own_state: bool = False
 
 
 @dataclass(frozen=True)

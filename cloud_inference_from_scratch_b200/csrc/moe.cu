@@ -9,14 +9,16 @@
 //              of the best groups can be chosen
 //   plan       counts per expert -> offsets; every (token, choice) pair gets a place in its expert's
 //              run of rows; runs are cut into tiles of 128 rows for the grouped products
-//   gate_up    rows gathered by place, times the expert's stacked gate and up matrices, SiLU(gate)*up
+//   gate_up    rows gathered by place, times the expert's stacked gate and up matrices, SiLU(gate)*up or another
+//              gated activation (glu.cuh); a pair's weight may multiply its row here instead of in the sum
 //   down       times the expert's down matrix, written to the pair's own row (float32)
-//   combine    y[t] = sum over the token's choices, in the order they were chosen, of weight * row
+//   combine    y[t] = sum over the token's choices, in the order they were chosen, of weight * row (or of row)
 //
 // The grouped products here run on the CUDA cores with float32 accumulation, one fused multiply-add
 // per k in ascending order: the 32-bit path's products, and what every shape can fall back on.  A
 // pair's row does not depend on which place it got, so the batch never changes a result.
 #include "common.cuh"
+#include "glu.cuh"
 
 #include <cfloat>
 
@@ -227,7 +229,7 @@ __global__ void __launch_bounds__(256)
 moe_grouped_simt_kernel(const T* __restrict__ a, const T* __restrict__ w0, const T* __restrict__ w1,
                         void* __restrict__ out, const int* __restrict__ place_to_pair,
                         const int* __restrict__ tiles, const int* __restrict__ tile_count, int top,
-                        int n_total, int k_total) {
+                        int n_total, int k_total, GluAct glu_act) {
   constexpr int kTileN = 64, kTileK = 16, kHalf = 64;
   static_assert(kRowTile == 2 * kHalf, "a block takes half a tile");
   __shared__ float a_tile[kTileK][kHalf + 4];
@@ -288,14 +290,14 @@ moe_grouped_simt_kernel(const T* __restrict__ a, const T* __restrict__ w0, const
   for (int i = 0; i < 4; ++i) {
     const int r = tm + i;
     if (r >= rows) continue;
+    const float weight = kGateUp && glu_act.weights ? glu_act.weights[place_to_pair[place0 + r]] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int gn = n0 + tn + j;
       if (gn >= n_total) continue;
       if constexpr (kGateUp) {
-        const float g = acc[i][j];
         reinterpret_cast<T*>(out)[(size_t)(place0 + r) * n_total + gn] =
-            from_float<T>(g / (1.f + expf(-g)) * acc_up[i][j]);
+            from_float<T>(glu(glu_act, acc[i][j], acc_up[i][j], weight));
       } else {
         reinterpret_cast<float*>(out)[(size_t)place_to_pair[place0 + r] * n_total + gn] = acc[i][j];
       }
@@ -341,7 +343,7 @@ __global__ void __launch_bounds__(256)
 moe_grouped_tc_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ w0,
                       const __nv_bfloat16* __restrict__ w1, void* __restrict__ out,
                       const int* __restrict__ place_to_pair, const int* __restrict__ tiles,
-                      const int* __restrict__ tile_count, int top, int n_total, int k_total, int interleaved) {
+                      const int* __restrict__ tile_count, int top, int n_total, int k_total, int interleaved, GluAct glu_act) {
   // interleaved (gate_up only): w0 holds [experts][2 * n_total][k], 16 gate rows, their 16 up rows, ...
   constexpr int kWRows = kGateUp ? 2 * kTcCols : kTcCols;
   constexpr int kNT = kGateUp ? 8 : 4;                    // 8-column accumulators of a warp
@@ -352,6 +354,7 @@ moe_grouped_tc_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* 
   WTile w_s = reinterpret_cast<WTile>(tc_smem + (size_t)kTcStages * kRowTile * kTcLd * sizeof(__nv_bfloat16));
   __shared__ int src_row[kRowTile];
   __shared__ int dst_row[kRowTile];
+  __shared__ float weight_of[kGateUp ? kRowTile : 1];
   pdl_wait();
   pdl_trigger();
   if ((int)blockIdx.y >= tile_count[0]) return;
@@ -363,6 +366,7 @@ moe_grouped_tc_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* 
       const int pair = place_to_pair[place0 + tid];
       src = kGateUp ? pair / top : place0 + tid;
       dst = kGateUp ? place0 + tid : pair;
+      if (kGateUp) weight_of[tid] = glu_act.weights ? glu_act.weights[pair] : 1.f;
     }
     src_row[tid] = src;
     dst_row[tid] = dst;
@@ -445,7 +449,7 @@ moe_grouped_tc_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* 
           if (gn >= n_total) continue;
           if constexpr (kGateUp) {
             const float g = acc[mt][nt][2 * half + e], u = acc[mt][4 + nt][2 * half + e];
-            reinterpret_cast<__nv_bfloat16*>(out)[(size_t)dst * n_total + gn] = __float2bfloat16_rn(g / (1.f + expf(-g)) * u);
+            reinterpret_cast<__nv_bfloat16*>(out)[(size_t)dst * n_total + gn] = __float2bfloat16_rn(glu(glu_act, g, u, weight_of[r]));
           } else {
             reinterpret_cast<float*>(out)[(size_t)dst * n_total + gn] = acc[mt][nt][2 * half + e];
           }
@@ -453,7 +457,8 @@ moe_grouped_tc_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* 
     }
 }
 
-// y[t][i] = sum_j weights[t][j] * rows[t * top + j][i], j ascending; float32 or activation type out.
+// y[t][i] = sum_j weights[t][j] * rows[t * top + j][i], j ascending (weights null: all ones); float32 or activation
+// type out.
 template <typename TOut>
 __global__ void moe_combine_kernel(const float* __restrict__ rows, const float* __restrict__ weights,
                                    TOut* __restrict__ y, int hidden, int top) {
@@ -463,7 +468,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ rows, const float* 
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     float total = 0.f;
     for (int j = 0; j < top; ++j)
-      total = fmaf(weights[(size_t)t * top + j], rows[((size_t)t * top + j) * hidden + i], total);
+      total = fmaf(weights ? weights[(size_t)t * top + j] : 1.f, rows[((size_t)t * top + j) * hidden + i], total);
     y[(size_t)t * hidden + i] = from_float<TOut>(total);
   }
 }
@@ -515,22 +520,24 @@ extern "C" int cie_moe_route(const void* x, const float* router, const float* co
   return 0;
 }
 
-// act: [pairs][ff] activation type, rows by place.  w_gate, w_up: [experts][ff][hidden].
+// act: [pairs][ff] activation type, rows by place.  w_gate, w_up: [experts][ff][hidden].  clamped, limit, slope,
+// shift, input_weights: see GluAct.
 extern "C" int cie_moe_gate_up_simt(const void* x, const void* w_gate, const void* w_up, void* act,
                                     const int* place_to_pair, const int* tiles, const int* tile_count,
-                                    int tokens, int top, int experts, int ff, int hidden, int dtype,
-                                    void* stream) {
+                                    int tokens, int top, int experts, int ff, int hidden, int clamped, float limit,
+                                    float slope, float shift, const float* input_weights, int dtype, void* stream) {
   if (tokens <= 0) return 0;
+  const GluAct glu_act{clamped, limit, slope, shift, input_weights};
   const int max_tiles = (tokens * top + kRowTile - 1) / kRowTile + experts;
   dim3 grid((ff + 63) / 64, 2 * max_tiles);
   if (dtype == kFloat32) {
     CIE_LAUNCH("moe_gate_up", (moe_grouped_simt_kernel<float, true>), grid, dim3(256), 0, (cudaStream_t)stream,
                (const float*)x, (const float*)w_gate, (const float*)w_up, act, place_to_pair, tiles, tile_count, top,
-               ff, hidden);
+               ff, hidden, glu_act);
   } else if (dtype == kBFloat16) {
     CIE_LAUNCH("moe_gate_up", (moe_grouped_simt_kernel<__nv_bfloat16, true>), grid, dim3(256), 0, (cudaStream_t)stream,
                (const __nv_bfloat16*)x, (const __nv_bfloat16*)w_gate, (const __nv_bfloat16*)w_up, act, place_to_pair,
-               tiles, tile_count, top, ff, hidden);
+               tiles, tile_count, top, ff, hidden, glu_act);
   } else {
     CIE_FAIL("moe_gate_up: unknown element type code %d", dtype);
   }
@@ -547,11 +554,11 @@ extern "C" int cie_moe_down_simt(const void* act, const void* w_down, float* row
   if (dtype == kFloat32) {
     CIE_LAUNCH("moe_down", (moe_grouped_simt_kernel<float, false>), grid, dim3(256), 0, (cudaStream_t)stream,
                (const float*)act, (const float*)w_down, (const float*)nullptr, (void*)rows, place_to_pair, tiles,
-               tile_count, top, hidden, ff);
+               tile_count, top, hidden, ff, GluAct{});
   } else if (dtype == kBFloat16) {
     CIE_LAUNCH("moe_down", (moe_grouped_simt_kernel<__nv_bfloat16, false>), grid, dim3(256), 0, (cudaStream_t)stream,
                (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, (const __nv_bfloat16*)nullptr, (void*)rows,
-               place_to_pair, tiles, tile_count, top, hidden, ff);
+               place_to_pair, tiles, tile_count, top, hidden, ff, GluAct{});
   } else {
     CIE_FAIL("moe_down: unknown element type code %d", dtype);
   }
@@ -563,7 +570,8 @@ extern "C" int cie_moe_down_simt(const void* act, const void* w_down, float* row
 // w_up null: w_gate holds both, [experts][2 ff][hidden], interleaved in blocks of 16 rows.
 extern "C" int cie_moe_gate_up_tc(const void* x, const void* w_gate, const void* w_up, void* act,
                                   const int* place_to_pair, const int* tiles, const int* tile_count,
-                                  int tokens, int top, int experts, int ff, int hidden, void* stream) {
+                                  int tokens, int top, int experts, int ff, int hidden, int clamped, float limit,
+                                  float slope, float shift, const float* input_weights, void* stream) {
   if (!w_up && ff % 16) CIE_FAIL("moe_gate_up_tc: interleaved weights need a multiple of 16 channels, got %d", ff);
   if (tokens <= 0) return 0;
   if (hidden % 8 || ff % 8) CIE_FAIL("moe_gate_up_tc: sizes %d / %d are no multiples of 8", hidden, ff);
@@ -578,7 +586,7 @@ extern "C" int cie_moe_gate_up_tc(const void* x, const void* w_gate, const void*
   }
   CIE_LAUNCH("moe_gate_up_tc", moe_grouped_tc_kernel<true>, grid, dim3(256), moe_tc_smem<true>(), (cudaStream_t)stream,
              (const __nv_bfloat16*)x, (const __nv_bfloat16*)w_gate, (const __nv_bfloat16*)w_up, act, place_to_pair,
-             tiles, tile_count, top, ff, hidden, w_up ? 0 : 1);
+             tiles, tile_count, top, ff, hidden, w_up ? 0 : 1, GluAct{clamped, limit, slope, shift, input_weights});
   return 0;
 }
 
@@ -598,7 +606,7 @@ extern "C" int cie_moe_down_tc(const void* act, const void* w_down, float* rows,
   }
   CIE_LAUNCH("moe_down_tc", moe_grouped_tc_kernel<false>, grid, dim3(256), moe_tc_smem<false>(), (cudaStream_t)stream,
              (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, (const __nv_bfloat16*)nullptr, (void*)rows,
-             place_to_pair, tiles, tile_count, top, hidden, ff, 0);
+             place_to_pair, tiles, tile_count, top, hidden, ff, 0, GluAct{});
   return 0;
 }
 

@@ -19,6 +19,7 @@
 // runs beside the other's products.  Every wait on an mbarrier is bounded.
 #include "blackwell.cuh"
 #include "common.cuh"
+#include "glu.cuh"
 
 CIE_DEFINE_LAST_ERROR()
 
@@ -66,6 +67,7 @@ struct GroupedArgs {
   int n;                   // output columns of a row (F or H)
   int k;
   int* err;
+  GluAct glu_act;          // gate_up
 };
 
 template <bool kGateUp, int BN>
@@ -148,6 +150,7 @@ __global__ void __launch_bounds__(128) moe_grouped_tcgen05_kernel(const __grid_c
     const uint32_t lane_base = tmem_base + ((uint32_t)(warp * 32) << 16);
     if constexpr (kGateUp) {
       bf16* dst_row = reinterpret_cast<bf16*>(a.out) + (size_t)(place0 + r) * a.n;
+      const float weight = live && a.glu_act.weights ? a.glu_act.weights[a.place_to_pair[place0 + r]] : 1.f;
 #pragma unroll 1
       for (int c0 = 0; c0 < BN; c0 += 32) {
         uint32_t gate[16], up[16];
@@ -159,19 +162,16 @@ __global__ void __launch_bounds__(128) moe_grouped_tcgen05_kernel(const __grid_c
           uint32_t packed[8];
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
-            const float g0 = __uint_as_float(gate[2 * j]), g1 = __uint_as_float(gate[2 * j + 1]);
-            const float v0 = g0 / (1.f + expf(-g0)) * __uint_as_float(up[2 * j]);
-            const float v1 = g1 / (1.f + expf(-g1)) * __uint_as_float(up[2 * j + 1]);
+            const float v0 = glu(a.glu_act, __uint_as_float(gate[2 * j]), __uint_as_float(up[2 * j]), weight);
+            const float v1 = glu(a.glu_act, __uint_as_float(gate[2 * j + 1]), __uint_as_float(up[2 * j + 1]), weight);
             __nv_bfloat162 pair = __floats2bfloat162_rn(v0, v1);
             packed[j] = *reinterpret_cast<uint32_t*>(&pair);
           }
           reinterpret_cast<uint4*>(dst_row + channel0)[0] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
           reinterpret_cast<uint4*>(dst_row + channel0)[1] = make_uint4(packed[4], packed[5], packed[6], packed[7]);
         } else {
-          for (int j = 0; j < 16 && channel0 + j < a.n; ++j) {
-            const float g = __uint_as_float(gate[j]);
-            dst_row[channel0 + j] = __float2bfloat16_rn(g / (1.f + expf(-g)) * __uint_as_float(up[j]));
-          }
+          for (int j = 0; j < 16 && channel0 + j < a.n; ++j)
+            dst_row[channel0 + j] = __float2bfloat16_rn(glu(a.glu_act, __uint_as_float(gate[j]), __uint_as_float(up[j]), weight));
         }
       }
     } else {
@@ -231,11 +231,12 @@ using namespace cie;
 
 // x: [tokens][hidden]; sorted: scratch [tokens * top][hidden]; w_gate_up: [experts][2 ff][hidden], gate
 // and up rows interleaved in blocks of 16; act: [tokens * top][ff], rows by place.  All bfloat16,
-// 16-byte aligned; hidden a multiple of 8, ff a multiple of 16.
+// 16-byte aligned; hidden a multiple of 8, ff a multiple of 16.  clamped, limit, slope, shift, input_weights: GluAct.
 extern "C" int cie_moe_gate_up_tcgen05(const void* x, void* sorted, const void* w_gate_up, void* act,
                                        const int* place_to_pair, const int* tiles, const int* tile_count,
-                                       int tokens, int top, int experts, int ff, int hidden, int row_tile,
-                                       int* err, void* stream) {
+                                       int tokens, int top, int experts, int ff, int hidden, int row_tile, int clamped,
+                                       float limit, float slope, float shift, const float* input_weights, int* err,
+                                       void* stream) {
   if (tokens <= 0) return 0;
   if (hidden % 8 || ff % 16) CIE_FAIL("moe_gate_up_tcgen05: sizes %d / %d", hidden, ff);
   if (row_tile != BM) CIE_FAIL("moe_gate_up_tcgen05: tiles of %d rows, this kernel takes %d", row_tile, BM);
@@ -254,7 +255,8 @@ extern "C" int cie_moe_gate_up_tcgen05(const void* x, void* sorted, const void* 
   if (!tensor_map_bf16(sorted, pairs, hidden, BM, &map_a) ||
       !tensor_map_bf16(w_gate_up, (long long)experts * 2 * ff, hidden, bn, &map_b))
     CIE_FAIL("moe_gate_up_tcgen05: cuTensorMapEncodeTiled failed");
-  GroupedArgs a = {act, place_to_pair, tiles, tile_count, 2 * ff, ff, hidden, err};
+  GroupedArgs a = {act, place_to_pair, tiles, tile_count, 2 * ff, ff, hidden, err,
+                   {clamped, limit, slope, shift, input_weights}};
   const int max_tiles = (pairs + BM - 1) / BM + experts;
   const dim3 grid((2 * ff + bn - 1) / bn, max_tiles);
   return bn == 256 ? launch_grouped<true, 256>(map_a, map_b, a, grid, s) : launch_grouped<true, 128>(map_a, map_b, a, grid, s);
@@ -276,7 +278,7 @@ extern "C" int cie_moe_down_tcgen05(const void* act, const void* w_down, float* 
   if (!tensor_map_bf16(act, pairs, ff, BM, &map_a) ||
       !tensor_map_bf16(w_down, (long long)experts * hidden, ff, bn, &map_b))
     CIE_FAIL("moe_down_tcgen05: cuTensorMapEncodeTiled failed");
-  GroupedArgs a = {rows, place_to_pair, tiles, tile_count, hidden, hidden, ff, err};
+  GroupedArgs a = {rows, place_to_pair, tiles, tile_count, hidden, hidden, ff, err, {}};
   const int max_tiles = (pairs + BM - 1) / BM + experts;
   const dim3 grid((hidden + bn - 1) / bn, max_tiles);
   cudaStream_t s = (cudaStream_t)stream;

@@ -28,7 +28,7 @@ class KVLayerView:
 @dataclass
 class LayerBinding:
     """What one schedule entry sees of the cache.  ``owns_cache`` False: it reads what an earlier
-    entry wrote and must write nothing.  ``state``: [request slots, *state shape] or None."""
+    entry wrote and must write nothing to its pages.  ``state``: [request slots, *state shape] or None."""
 
     entry: int
     owns_cache: bool

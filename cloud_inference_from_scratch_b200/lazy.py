@@ -99,11 +99,11 @@ class NormedInput:
 
 class NormedUpdate:
     """A result ``y`` [T, H] that joins the residual stream RMS-normalised: ``x <- x + gain * y / rms(y)``, the root mean
-    square over the whole row with ``eps`` inside.  The norm that reads the stream next applies it in its own kernel,
-    in float32."""
+    square over the whole row with ``eps`` inside; ``centred``: layer-normalised, ``gain * (y - mean(y)) / sqrt(mean((y -
+    mean(y))^2) + eps)``.  Whoever reads the stream next applies it in its own kernel, in float32."""
 
-    def __init__(self, y: Any, gain: Any, eps: float) -> None:
-        self.y, self.gain, self.eps = y, gain, float(eps)
+    def __init__(self, y: Any, gain: Any, eps: float, centred: bool = False) -> None:
+        self.y, self.gain, self.eps, self.centred = y, gain, float(eps), bool(centred)
 
     @property
     def shape(self) -> tuple[int, ...]:
@@ -112,11 +112,13 @@ class NormedUpdate:
 
 class WeightedTerms:
     """A weighted sum that has not been taken yet: row t is ``sum_j weights[t, j] * terms[t, j]``, with ``terms`` float32
-    [T, count * H] (the ``count`` terms of a row side by side) and ``weights`` float32 [T, count].  The norm that reads the
-    stream next takes it in its own kernel, in float32, in ascending order."""
+    [T, count * H] (the ``count`` terms of a row side by side) and ``weights`` float32 [T, count] (None: all ones; then
+    ``count`` is given), plus ``extra[t]`` (float32 [T, H]) if there is one.  Whoever reads the stream next takes it in its
+    own kernel, in float32, in ascending order."""
 
-    def __init__(self, terms: Any, weights: Any) -> None:
-        self.terms, self.weights, self.count = terms, weights, int(weights.shape[1])
+    def __init__(self, terms: Any, weights: Any, count: int = 0, extra: Any = None) -> None:
+        self.terms, self.weights, self.count = terms, weights, int(count or weights.shape[1])
+        self.extra = extra
 
     @property
     def shape(self) -> tuple[int, ...]:
@@ -134,6 +136,28 @@ class PendingNorm:
     @property
     def shape(self) -> tuple[int, ...]:
         return tuple(self.residual.shape)
+
+
+class PendingStream:
+    """The stream as a sublayer reads it where no norm stands in front, with the update that still has to join it.
+    Whoever takes this instead of a tensor (``takes_pending_stream``) lets it join in its own first kernel."""
+
+    def __init__(self, residual: Any, update: Any) -> None:
+        self.residual, self.update = residual, update
+
+    @property
+    def shape(self) -> tuple[int, ...]:
+        return tuple(self.residual.shape)
+
+
+class DepthUpdate:
+    """A layer's last update together with what the layer's result means for the stream.  With ``row = base + update``
+    (``base`` None: the stream itself) the row is kept as state ``place`` of ``history`` [T, states * H] (None: it is
+    not kept), and the stream becomes ``sum_(j < place) share[j] * history_j + share[place] * row``, or the row itself
+    if ``share`` is None."""
+
+    def __init__(self, update: Any, base: Any, history: Any, place: int, share: Any) -> None:
+        self.update, self.base, self.history, self.place, self.share = update, base, history, int(place), share
 
 
 class StreamUpdate:

@@ -65,12 +65,14 @@ class LayerParts:
 @dataclass(frozen=True)
 class CacheNeed:
     """What one schedule entry needs of the cache manager (``owner`` is the entry whose
-    cache it uses: itself, or the earlier entry it reads)."""
+    pages it uses: itself, or the earlier entry it reads; ``state_owner`` the same for the
+    per-request state)."""
 
     entry: int
     owner: int
     pages: CacheSpec | None
     state: StateSpec | None
+    state_owner: int
 
 
 class DecoderModel:
@@ -154,11 +156,11 @@ class DecoderModel:
             owner = index if entry.reads_cache_of is None else entry.reads_cache_of
             pages = keeper.cache_spec() if keeper is not None and hasattr(keeper, "cache_spec") else None
             state = keeper.state_spec() if keeper is not None and hasattr(keeper, "state_spec") else None
-            needs.append(CacheNeed(index, owner, pages, state))
+            needs.append(CacheNeed(index, owner, pages, state, index if entry.own_state else owner))
         for need in needs:
             if need.owner != need.entry:
                 owner = needs[need.owner]
-                if (owner.pages, owner.state) != (need.pages, need.state):
+                if owner.pages != need.pages or (need.state_owner == need.owner and owner.state != need.state):
                     raise ValueError(
                         f"schedule entry {need.entry} reads the cache of entry {need.owner}, "
                         "whose mixer keeps a different kind of cache"

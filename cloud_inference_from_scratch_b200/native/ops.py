@@ -15,7 +15,7 @@ import os
 from ctypes import c_float, c_int, c_void_p
 from typing import Any
 
-from ..lazy import Accumulated, GateUpWeight, NormedInput, NormedUpdate, Partials, ResidualSink, StreamUpdate, WeightedTerms  # noqa: F401  (re-exported)
+from ..lazy import Accumulated, DepthUpdate, GateUpWeight, NormedInput, NormedUpdate, Partials, ResidualSink, StreamUpdate, WeightedTerms  # noqa: F401  (re-exported)
 from .build import load_library
 
 F32, BF16 = 0, 1
@@ -123,6 +123,7 @@ class Ops:
         self._moe_lib = None
         self._grouped_lib = None
         self._ssd_lib = None
+        self._stream_step_lib = None
         self._sample = None   # sampling.cu is built when something is first sampled
         self._tensor_gemm = None
         self._fold_gemm_held = None
@@ -631,9 +632,13 @@ class Ops:
         weights, gain, eps (and what must stay alive until the launch)."""
         gain, eps, weights = None, 0.0, None
         if isinstance(update, NormedUpdate):
+            if update.centred:
+                raise KernelError("group_norm: a layer-normalised update")
             gain, eps, update = update.gain, update.eps, update.y
         if isinstance(update, Accumulated):
             raise KernelError("group_norm: an update that is already in the stream")
+        if isinstance(update, WeightedTerms) and update.extra is not None:
+            raise KernelError("group_norm: a weighted sum with one more term")
         if isinstance(update, Partials) and (update.splits == 0 or update.bias is not None):
             update = self.resolve(update, self.torch.empty(update.shape, dtype=self.torch.float32, device=self.device))
         if update is None:
@@ -698,6 +703,79 @@ class Ops:
         self.launches += 1
         self._side_gate(_ptr(z), _ptr(token_ids), _ptr(table), table.shape[1], table.shape[0], int(column), _ptr(out),
                         out.shape[0], out.shape[1], self._code_of(out), _ptr(self.error_word), self.stream)
+
+    # ------------------------------------------------------------------ a stream with normalised updates
+    def _load_stream_step(self) -> None:
+        if self._stream_step_lib is None:
+            v, i, f, ll = c_void_p, c_int, c_float, ctypes.c_longlong
+            lib = _Lib(load_library("stream_step.cu"))
+            self._stream_advance = lib.function(
+                "cie_stream_advance",
+                [v, ll, v, i, ll, ll, v, v, v, f, i, v, ll, i, v, v, ll, v, v, i, v, i, i, v, v, ll, v, v, v, v, i, i, v, f,
+                 i, v, v])
+            self.stream_step_max_width = int(lib.handle.cie_stream_step_max_width())
+            self._stream_step_lib = lib
+
+    def require_stream_step(self) -> int:
+        """Builds, at model set-up, the kernels of ``advance``; returns the widest row they take."""
+        self._load_stream_step()
+        return self.stream_step_max_width
+
+    def advance(self, residual: Any, pending: Any, out: Any, rows: Any = None, write: bool = True,
+                shift: "tuple[Any, Any] | None" = None, norm: "tuple[Any, float] | None" = None, ctx: Any = None) -> None:
+        """What is pending joins the float32 stream, and ``out`` gets the stream's rows x, rounded once: as they are;
+        with ``shift`` = (share [H], state [slots, >= H] float32) as ``x_t + (x_(t - 1) - x_t) * share`` within each
+        request of ``ctx`` (its state stands in for the row before the step's first, and becomes the row of its last
+        token); with ``norm`` = (gain, eps) as their layer norm.  ``pending``: None, float32 terms (a tensor,
+        ``Partials``, ``WeightedTerms``), a ``NormedUpdate`` of those, or a ``DepthUpdate``.  With ``rows`` only those
+        rows are read and nothing but ``out`` is written; ``write`` False leaves the stream as it was (a ``DepthUpdate``
+        still keeps its state)."""
+        self._flush()
+        self._load_stream_step()
+        count, hidden = out.shape
+        base, history, place, share = residual, None, 0, None
+        if isinstance(pending, DepthUpdate):
+            base = residual if pending.base is None else pending.base
+            history, place, share, pending = pending.history, pending.place, pending.share, pending.update
+        gain, eps, kind = None, 0.0, 0
+        if isinstance(pending, NormedUpdate):
+            gain, eps, kind, pending = pending.gain, pending.eps, 2 if pending.centred else 1, pending.y
+        if isinstance(pending, Accumulated):
+            raise KernelError("advance: an update that is already in the stream")
+        extra = weights = data = None
+        terms = stride = row_stride = 0
+        if isinstance(pending, Partials) and (pending.splits == 0 or pending.bias is not None):
+            pending = self.resolve(pending, self.torch.empty(pending.shape, dtype=self.torch.float32, device=self.device))
+        if isinstance(pending, WeightedTerms):
+            data, terms, stride, row_stride = pending.terms, pending.count, hidden, pending.count * hidden
+            weights, extra = pending.weights, pending.extra
+        elif isinstance(pending, Partials):
+            data, terms, stride, row_stride = pending.data, pending.splits, pending.stride, hidden
+        elif pending is not None:
+            data, terms, row_stride = pending if pending.dtype == self.torch.float32 else pending.float(), 1, hidden
+        keep, history_stride = None, 0
+        if history is not None:
+            history_stride = history.stride(0)
+            if rows is None:
+                keep = history.data_ptr() + 4 * place * hidden
+        # x is what the stream holds already where nothing joins it
+        stream = residual if rows is None and write and (data is not None or share is not None) else None
+        out_kind, share_vector, state, state_stride, slots = 0, None, None, 0, 0
+        singles = True
+        if shift is not None:
+            out_kind, (share_vector, state) = 1, shift
+            state_stride, slots = state.stride(0), state.shape[0]
+            singles = count == ctx.num_requests and ctx.num_single == ctx.num_requests
+        elif norm is not None:
+            out_kind = 2
+        self.launches += 1 if singles else 2
+        request = (_ptr(ctx.query_start), _ptr(ctx.request_of_token), _ptr(ctx.slots), _ptr(ctx.request_active)) if shift is not None else (None,) * 4
+        self._stream_advance(_ptr(base), base.stride(0), _ptr(data), terms, stride, row_stride, _ptr(weights), _ptr(extra),
+                             _ptr(gain), float(eps), kind, _ptr(history), history_stride, place if share is not None else 0,
+                             _ptr(share), keep, history_stride, _ptr(stream), _ptr(out), out_kind, _ptr(rows), count, hidden,
+                             _ptr(share_vector), _ptr(state), state_stride, *request, slots, 1 if singles else 0,
+                             _ptr(norm[0]) if norm is not None else None, float(norm[1]) if norm is not None else 0.0,
+                             self._code_of(out), _ptr(self.error_word), self.stream)
 
     # ------------------------------------------------------------------ state-space recurrence
     def _load_ssd(self) -> None:
@@ -1204,10 +1282,10 @@ class Ops:
             v, i, f = c_void_p, c_int, c_float
             lib = _Lib(load_library("moe.cu"))
             self._moe_route = lib.function("cie_moe_route", [v, v, v, v, v, v, v, v, v, v, v, i, i, i, i, i, v, i, i, i, i, f, i, v])
-            self._moe_gate_up_simt = lib.function("cie_moe_gate_up_simt", [v, v, v, v, v, v, v, i, i, i, i, i, i, v])
+            self._moe_gate_up_simt = lib.function("cie_moe_gate_up_simt", [v, v, v, v, v, v, v, i, i, i, i, i, i, f, f, f, v, i, v])
             self._moe_down_simt = lib.function("cie_moe_down_simt", [v, v, v, v, v, v, i, i, i, i, i, i, v])
             self._moe_combine = lib.function("cie_moe_combine", [v, v, v, i, i, i, i, v])
-            self._moe_gate_up_tc = lib.function("cie_moe_gate_up_tc", [v, v, v, v, v, v, v, i, i, i, i, i, v])
+            self._moe_gate_up_tc = lib.function("cie_moe_gate_up_tc", [v, v, v, v, v, v, v, i, i, i, i, i, i, f, f, f, v, v])
             self._moe_down_tc = lib.function("cie_moe_down_tc", [v, v, v, v, v, v, i, i, i, i, i, v])
             self.moe_row_tile = int(lib.handle.cie_moe_row_tile())
             self._moe_lib = lib
@@ -1215,10 +1293,10 @@ class Ops:
 
     def _load_moe_tcgen05(self) -> None:
         if self._moe_tcgen05_lib is None:
-            v, i = c_void_p, c_int
+            v, i, f = c_void_p, c_int, c_float
             lib = _Lib(load_library("moe_tcgen05.cu"))
             self._moe_gate_up_tcgen05 = lib.function(
-                "cie_moe_gate_up_tcgen05", [v, v, v, v, v, v, v, i, i, i, i, i, i, v, v])
+                "cie_moe_gate_up_tcgen05", [v, v, v, v, v, v, v, i, i, i, i, i, i, i, f, f, f, v, v, v])
             self._moe_down_tcgen05 = lib.function(
                 "cie_moe_down_tcgen05", [v, v, v, v, v, v, i, i, i, i, i, i, v, v])
             self._moe_tcgen05_lib = lib
@@ -1238,7 +1316,8 @@ class Ops:
     def routed_experts(self, x: Any, router: Any, correction: Any, w_gate: Any, w_up: Any, w_down: Any,
                        top: int, renormalize: bool, out: Any, workspace: Any, router_bias: Any = None,
                        chosen_softmax: bool = False, sigmoid: bool = False, groups: tuple[int, int] = (1, 1),
-                       norm_floor: float = 0.0, defer: bool = False) -> Any:
+                       norm_floor: float = 0.0, defer: bool = False,
+                       activation: tuple[float, float, float] | None = None, weight_inputs: bool = False) -> Any:
         """out[t] = sum over the ``top`` chosen experts e of score_e * down_e(SiLU(gate_e x) * up_e x).
         ``router`` float32 [E, H]; ``w_gate``/``w_up`` [E, F, H], or ``w_up`` None and ``w_gate`` the
         interleaved [E, 2F, H] of ``interleave_gate_up``; ``w_down`` [E, H, F]; ``out`` float32 or the
@@ -1247,9 +1326,13 @@ class Ops:
         ``sigmoid``: scores are sigmoids of the logits; ``groups`` = (count, keep): experts form equal groups of
         neighbours and only those of the ``keep`` groups whose two largest choice scores have the largest sums can
         be chosen; ``norm_floor`` is added to the sum that ``renormalize`` divides by.  ``defer``: the weighted sum is
-        left to the kernel that reads the stream next (``out`` is not written; ``WeightedTerms`` is returned)."""
+        left to the kernel that reads the stream next (``out`` is not written; ``WeightedTerms`` is returned).
+        ``activation`` (limit, slope, shift): gate capped at ``limit``, up clamped to +-``limit``, then gate *
+        sigmoid(slope * gate) * (up + shift).  ``weight_inputs``: score_e multiplies the expert's input instead of its
+        output (out[t] = sum of e(score_e * x))."""
         self._flush()
         self._load_moe()
+        glu = (1, *(float(number) for number in activation)) if activation is not None else (0, 0.0, 1.0, 0.0)
         torch = self.torch
         tokens, hidden = x.shape
         experts, ff = w_gate.shape[0], w_gate.shape[1] // (2 if w_up is None else 1)
@@ -1272,6 +1355,8 @@ class Ops:
                         _ptr(offsets), _ptr(cursors), _ptr(place_to_pair), _ptr(tiles), _ptr(tile_count), tokens,
                         hidden, experts, top, 1 if renormalize else 0, _ptr(router_bias), 1 if chosen_softmax else 0,
                         1 if sigmoid else 0, groups[0], groups[1], float(norm_floor), code, self.stream)
+        glu = (*glu, _ptr(weights) if weight_inputs else None)
+        out_weights = None if weight_inputs else weights
         aligned = (x.data_ptr() | w_gate.data_ptr() | w_down.data_ptr() | act.data_ptr()) % 16 == 0
         if w_up is None and not (code == BF16 and aligned):
             raise KernelError("routed_experts: interleaved gate/up weights are for aligned bfloat16 operands")
@@ -1282,7 +1367,7 @@ class Ops:
             gathered = workspace.get("moe.sorted", tokens, top * hidden, self.dtype)
             self._moe_gate_up_tcgen05(_ptr(x), _ptr(gathered), _ptr(w_gate), _ptr(act), _ptr(place_to_pair),
                                       _ptr(tiles), _ptr(tile_count), tokens, top, experts, ff, hidden,
-                                      self.moe_row_tile, _ptr(self.error_word), self.stream)
+                                      self.moe_row_tile, *glu, _ptr(self.error_word), self.stream)
             self._moe_down_tcgen05(_ptr(act), _ptr(w_down), _ptr(rows), _ptr(place_to_pair), _ptr(tiles),
                                    _ptr(tile_count), tokens, top, experts, ff, hidden, self.moe_row_tile,
                                    _ptr(self.error_word), self.stream)
@@ -1291,18 +1376,18 @@ class Ops:
                 and (w_up is None or (os.environ.get("CIE_MOE_TC", "1") != "0" and w_up.data_ptr() % 16 == 0))):
             # bfloat16 on the tensor cores (mma.sync, float32 accumulators)
             self._moe_gate_up_tc(_ptr(x), _ptr(w_gate), _ptr(w_up), _ptr(act), _ptr(place_to_pair), _ptr(tiles),
-                                 _ptr(tile_count), tokens, top, experts, ff, hidden, self.stream)
+                                 _ptr(tile_count), tokens, top, experts, ff, hidden, *glu, self.stream)
             self._moe_down_tc(_ptr(act), _ptr(w_down), _ptr(rows), _ptr(place_to_pair), _ptr(tiles),
                               _ptr(tile_count), tokens, top, experts, ff, hidden, self.stream)
         else:
             self._moe_gate_up_simt(_ptr(x), _ptr(w_gate), _ptr(w_up), _ptr(act), _ptr(place_to_pair), _ptr(tiles),
-                                   _ptr(tile_count), tokens, top, experts, ff, hidden, code, self.stream)
+                                   _ptr(tile_count), tokens, top, experts, ff, hidden, *glu, code, self.stream)
             self._moe_down_simt(_ptr(act), _ptr(w_down), _ptr(rows), _ptr(place_to_pair), _ptr(tiles),
                                 _ptr(tile_count), tokens, top, experts, ff, hidden, code, self.stream)
         if defer:
             self.launches -= 1
-            return WeightedTerms(rows, weights)
-        self._moe_combine(_ptr(rows), _ptr(weights), _ptr(out), tokens, hidden, top, self._code_of(out), self.stream)
+            return WeightedTerms(rows, out_weights, count=top)
+        self._moe_combine(_ptr(rows), _ptr(out_weights), _ptr(out), tokens, hidden, top, self._code_of(out), self.stream)
         return out
 
     def stream_plan(self, m: int, n: int, k: int, allow_partials: bool) -> tuple[int, int] | None:

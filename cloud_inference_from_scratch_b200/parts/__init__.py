@@ -1,6 +1,6 @@
 from . import (  # noqa: F401  (registers the built-in parts)
     attention, block, connection, delta, gated_delta, gla, input_conv, latent, lightning, mamba2, matrix_memory, mlp,
-    norm, rotary, routed, side_by_side, token_side,
+    norm, rotary, routed, side_by_side, token_shift, token_side,
 )
 from .base import (
     Block,

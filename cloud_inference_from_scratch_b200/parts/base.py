@@ -37,7 +37,7 @@ class TensorSpec:
     """A tensor a part reads from the weight files.
 
     ``init`` is how the random-weights mode fills it: "normal" N(0, std), "gain"
-    1 + N(0, std), "eye" identity + N(0, std) (a square matrix), "zeros".  ``role`` "matrix" tensors are held in the compute dtype
+    1 + N(0, std), "mean" 1 / (number of elements) + N(0, std), "eye" identity + N(0, std) (a square matrix), "zeros".  ``role`` "matrix" tensors are held in the compute dtype
     (bfloat16 unless the whole run is 32-bit); "vector" tensors (norm gains, biases)
     are held in float32, which keeps a 32-bit stored tensor as it is and widens a
     bfloat16 one without loss; "table" tensors are integer tables held as int32.

@@ -1,4 +1,4 @@
-"""Pre-norm residual arrangement of one layer.
+"""Arrangements of one layer's parts around the residual stream.  The first and plainest, pre-norm:
 
 ``h = h + mixer(norm1(h)); h = h + feed_forward(norm2(h))`` (src/cloud_engine/model.py:212-220).
 The residual stream is float32 and each add is fused into the norm that follows it, so
@@ -139,3 +139,50 @@ class ParallelResidual(Block):
 
 
 register_part("block", "parallel_residual", ParallelResidual, replace=True)
+
+
+class PostNormResidual(Block):
+    """Each sublayer reads the stream itself and its RESULT is normalised: ``x <- x + norm1(mixer(x))``, then
+    ``x <- x + norm2(feed_forward(x))`` if the layer has a feed-forward.  An ``average`` part (a ``depth_average``
+    connection), if there is one, decides what goes on to the next layer.  Updates are not added by the norms but by
+    whoever reads the stream next, in the kernel that makes its rows (``Ops.advance``)."""
+
+    slots = ("mixer", "mixer_norm")
+
+    def __init__(self, parts, **params) -> None:
+        super().__init__(parts, **params)
+        if ("feed_forward" in parts) != ("feed_forward_norm" in parts):
+            raise ValueError("PostNormResidual: a feed-forward and its norm come together or not at all")
+
+    def _rows(self, residual, pending, runtime, write):
+        rows = runtime.workspace.get("norm.out", residual.shape[0], residual.shape[1], runtime.dtype)
+        runtime.ops.advance(residual, pending, rows, write=write)
+        return rows
+
+    def forward(self, residual, pending, ctx, binding):
+        from ..lazy import PendingStream
+
+        ctx.residual_sink = None           # a sublayer's result is normalised before it joins the stream
+        runtime = self.mixer.runtime
+        average = self.parts.get("average")
+        history = average.history(residual.shape[0]) if average is not None else None
+        if average is not None:
+            pending = average.entering(pending, history)
+        if getattr(self.mixer, "takes_pending_stream", False):
+            x = PendingStream(residual, pending)
+        else:
+            x = self._rows(residual, pending, runtime, True)
+        update = self.mixer_norm.of_update(self.mixer.forward(x, ctx, binding))
+        feed_forward = self.parts.get("feed_forward")
+        if feed_forward is not None:
+            if average is not None:
+                x = self._rows(residual, average.midway(update, history), runtime, False)
+            else:
+                x = self._rows(residual, update, runtime, True)
+            update = self.feed_forward_norm.of_update(feed_forward.forward(x, ctx))
+        if average is None:
+            return update
+        return average.leaving(update, history, feed_forward is not None)
+
+
+register_part("block", "postnorm_residual", PostNormResidual, replace=True)

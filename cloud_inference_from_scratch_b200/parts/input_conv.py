@@ -19,25 +19,22 @@ from ..lazy import PendingNorm
 from .base import Mixer, StateSpec, TensorSpec, build_part, register_part
 
 
-class InputConvolution(Mixer):
-    takes_pending_norm = True
+class InputState(Mixer):
+    """A mixer around an inner one that changes what the inner mixer reads with the help of earlier tokens' rows, which
+    it keeps as per-request state of ``kept_floats`` float32 numbers behind the inner mixer's own in the request's slot.
+    Where the inner mixer keeps its pages is the inner mixer's business."""
 
-    def __init__(self, hidden_size: int, taps: int, inner: PartSpec, name: str = "weight") -> None:
-        if taps < 1:
-            raise ValueError("the input convolution needs at least one tap")
-        self.hidden_size = int(hidden_size)
-        self.taps = int(taps)
-        self.name = str(name)
+    def __init__(self, inner: PartSpec, kept_floats: int) -> None:
         self.inner = build_part("mixer", inner)
         self.inner_prefix = inner.prefix
         kept = self.inner.state_spec()
         if kept is not None and not getattr(self.inner, "takes_state_views", False):
-            raise ValueError(f"input convolution: mixer {inner.kind!r} does not take its state as a view of a wider slot")
+            raise ValueError(f"{type(self).__name__}: mixer {inner.kind!r} does not take its state as a view of a wider slot")
         if kept is not None and kept.dtype != "float32":
-            raise ValueError("input convolution: the inner state must be float32")
+            raise ValueError(f"{type(self).__name__}: the inner state must be float32")
         # rounded up to whole 16-byte pieces, so that both parts of a slot are aligned
         self.inner_floats = -(-math.prod(kept.shape) // 4) * 4 if kept is not None else 0
-        self.history_floats = (self.taps - 1) * self.hidden_size
+        self.kept_floats = int(kept_floats)
         self.state_in_graphs = kept is None or self.inner.state_in_graphs
         self.kernels_through_ops = self.inner.kernels_through_ops
 
@@ -48,34 +45,60 @@ class InputConvolution(Mixer):
         return self.inner.cache_spec()
 
     def state_spec(self):
-        floats = self.inner_floats + -(-self.history_floats // 4) * 4
+        floats = self.inner_floats + -(-self.kept_floats // 4) * 4
         return StateSpec((floats,), "float32") if floats else None
+
+    def own_tensor_specs(self) -> dict[str, TensorSpec]:
+        raise NotImplementedError
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         specs = {self.inner_prefix + name: spec for name, spec in self.inner.tensor_specs().items()}
-        specs[self.name] = TensorSpec((self.hidden_size, self.taps), role="vector")
+        specs.update(self.own_tensor_specs())
         return specs
 
     def bind(self, tensors, runtime) -> None:
         self.runtime = runtime
+        self.inner.bind({name: tensors[self.inner_prefix + name] for name in self.inner.tensor_specs()}, runtime)
+
+    def kept(self, binding):
+        """The view of every slot's part that this wrapper keeps (None: nothing)."""
+        return binding.state[:, self.inner_floats:] if self.kept_floats else None
+
+    def run_inner(self, x, ctx, binding):
+        from dataclasses import replace
+
+        inner = binding.state[:, : self.inner_floats] if self.inner_floats else None
+        return self.inner.forward(x, ctx, replace(binding, state=inner))
+
+
+class InputConvolution(InputState):
+    takes_pending_norm = True
+
+    def __init__(self, hidden_size: int, taps: int, inner: PartSpec, name: str = "weight") -> None:
+        if taps < 1:
+            raise ValueError("the input convolution needs at least one tap")
+        self.hidden_size = int(hidden_size)
+        self.taps = int(taps)
+        self.name = str(name)
+        super().__init__(inner, (self.taps - 1) * self.hidden_size)
+
+    def own_tensor_specs(self) -> dict[str, TensorSpec]:
+        return {self.name: TensorSpec((self.hidden_size, self.taps), role="vector")}
+
+    def bind(self, tensors, runtime) -> None:
         longest = runtime.ops.require_grouped()
         if self.taps > longest:
             raise ValueError(f"the input convolution takes up to {longest} taps, got {self.taps}")
-        self.inner.bind({name: tensors[self.inner_prefix + name] for name in self.inner.tensor_specs()}, runtime)
+        super().bind(tensors, runtime)
         self.weight = tensors[self.name].float().contiguous()
 
     def forward(self, x, ctx, binding):
-        from dataclasses import replace
-
         if not isinstance(x, PendingNorm):
             raise TypeError("the input convolution begins with the norm in front of it; use a norm that can be handed on")
         rt = self.runtime
         out = rt.workspace.get("norm.out", x.shape[0], self.hidden_size, rt.dtype)
-        state = binding.state
-        history = state[:, self.inner_floats:] if self.history_floats else None
-        rt.ops.group_norm_conv(x.residual, x.update, x.gain, x.eps, x.groups, self.weight, history, out, ctx)
-        inner = state[:, : self.inner_floats] if self.inner_floats else None
-        return self.inner.forward(out, ctx, replace(binding, state=inner))
+        rt.ops.group_norm_conv(x.residual, x.update, x.gain, x.eps, x.groups, self.weight, self.kept(binding), out, ctx)
+        return self.run_inner(out, ctx, binding)
 
 
 register_part("mixer", "input_conv", InputConvolution, replace=True)

@@ -45,7 +45,7 @@ register_part("feed_forward", "swiglu", SwiGLU, replace=True)
 
 
 class ClampedGLU(FeedForward):
-    """Gated feed-forward with biases, a capped gate and a shifted up branch:
+    """Gated feed-forward with a capped gate and a shifted up branch (``bias=False``: without the biases):
     ``g = min(W_gate x + b_gate, limit)``, ``u = clamp(W_up x + b_up, -limit, limit)``,
     ``y = g * sigmoid(slope * g) * (u + shift)``, result ``W_down y + b_down``.  Gate and up are one
     stacked product with float32 results; biases, bounds and activation run in float32 in one kernel.
@@ -53,29 +53,31 @@ class ClampedGLU(FeedForward):
     ``up.b``, ``down``, ``down.b``."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, limit: float, slope: float = 1.702,
-                 shift: float = 1.0) -> None:
+                 shift: float = 1.0, bias: bool = True) -> None:
         self.hidden_size = int(hidden_size)
         self.intermediate_size = int(intermediate_size)
         self.limit = float(limit)
         self.slope = float(slope)
         self.shift = float(shift)
+        self.bias = bool(bias)
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         inter, hidden = self.intermediate_size, self.hidden_size
-        return {
-            "gate": TensorSpec((inter, hidden)), "gate.b": TensorSpec((inter,), role="vector"),
-            "up": TensorSpec((inter, hidden)), "up.b": TensorSpec((inter,), role="vector"),
-            "down": TensorSpec((hidden, inter)), "down.b": TensorSpec((hidden,), role="vector"),
-        }
+        specs = {"gate": TensorSpec((inter, hidden)), "up": TensorSpec((inter, hidden)),
+                 "down": TensorSpec((hidden, inter))}
+        if self.bias:
+            specs.update({"gate.b": TensorSpec((inter,), role="vector"), "up.b": TensorSpec((inter,), role="vector"),
+                          "down.b": TensorSpec((hidden,), role="vector")})
+        return specs
 
     def bind(self, tensors, runtime) -> None:
         import torch
 
         self.runtime = runtime
         self.w_gate_up = runtime.ops.prepare_weight(torch.cat([tensors["gate"], tensors["up"]]))
-        self.b_gate_up = torch.cat([tensors["gate.b"], tensors["up.b"]]).contiguous()
+        self.b_gate_up = torch.cat([tensors["gate.b"], tensors["up.b"]]).contiguous() if self.bias else None
         self.w_down = runtime.ops.prepare_weight(tensors["down"])
-        self.b_down = tensors["down.b"].contiguous()
+        self.b_down = tensors["down.b"].contiguous() if self.bias else None
 
     def forward(self, x, ctx):
         import torch

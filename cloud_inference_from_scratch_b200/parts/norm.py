@@ -8,7 +8,7 @@ the same kernel, and the result is rounded once to the compute dtype.
 
 from __future__ import annotations
 
-from ..lazy import Accumulated, NormedInput, PendingNorm
+from ..lazy import Accumulated, DepthUpdate, NormedInput, NormedUpdate, PendingNorm
 from .base import Norm, TensorSpec, register_part
 
 
@@ -57,6 +57,10 @@ class RMSNorm(Norm):
             return NormedInput(update, self.eps, materialize=lambda: self.forward(residual, None, ctx))
         return self.forward(residual, update, ctx)
 
+    def of_update(self, y):
+        """The norm of a sublayer's result that has not joined the stream yet."""
+        return NormedUpdate(y, self.weight, self.eps)
+
 
 register_part("norm", "rmsnorm", RMSNorm, replace=True)
 
@@ -95,9 +99,22 @@ class LayerNorm(Norm):
         count = residual.shape[0] if rows is None else rows.shape[0]
         out = rt.workspace.get("norm.out" if rows is None else "norm.rows", count,
                                self.hidden_size, rt.dtype, per_request=rows is not None)
+        if isinstance(update, (DepthUpdate, NormedUpdate)):
+            if self.bias is not None or self.update_scale != 1.0:
+                raise ValueError("layer norm: a normalised update joins the stream as it is, before a norm without bias")
+            if rows is None:
+                raise ValueError("layer norm: behind a normalised update only chosen rows are normalised")
+            rt.ops.advance(residual, update, out, rows=rows, norm=(self.weight, self.eps))
+            return out
         rt.ops.add_layernorm(residual, update, self.weight, self.bias, self.eps, out, rows,
                              update_scale=self.update_scale)
         return out
+
+    def of_update(self, y):
+        """The norm of a sublayer's result that has not joined the stream yet."""
+        if self.bias is not None or self.update_scale != 1.0:
+            raise ValueError("layer norm: the norm of an update has no bias and no factor")
+        return NormedUpdate(y, self.weight, self.eps, centred=True)
 
 
 register_part("norm", "layernorm", LayerNorm, replace=True)
