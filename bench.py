@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200, random weights.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl own|reference]
-                    [--config 3b|7b-mixed|14b-pressure|zisesun|lodalix|lazilorn|bilipel|sutuvik] [--quick]
+                    [--config 3b|7b-mixed|14b-pressure|zisesun|lodalix|lazilorn|bilipel|sutuvik|bozevik] [--quick]
 
 Prints ONE JSON line.  The default configuration is the Qwen2.5-3B shape: a "step" is one decode
 step of a batch of requests whose prompts (2,048 random tokens each) were prefilled before;
@@ -48,6 +48,12 @@ of 256 and 512 tokens, and (unless ``--quick``) the two other benchmark configur
   denominator; mixed values; an input convolution in front of every mixer; experts chosen from the best groups; a
   token side input) at two sizes, beside the Qwen2 dense shape of equal width, layer count, head count and active
   feed-forward size and beside the Zisesun configuration of that size, measured the same way.
+
+* ``bozevik``: the Bozevik design (latent attention on rows moved towards the token before, every other layer on the
+  latent of the layer before it; layer norms on the sublayers' results; an average over depth after every layer; a
+  clamped gated feed-forward, dense or routed with weighted inputs and a shared expert) at two sizes, beside the Qwen2
+  dense shape of equal width, layer count, head count and active feed-forward size and beside the Lodalix
+  configuration of that size, measured the same way.
 
 ``check`` compares, at the full 36 layers, the logits of the bfloat16 generation path with the
 32-bit path of the same weights (``engine/check.py``).  ``--config`` prints the line of one of the
@@ -711,7 +717,34 @@ SUTUVIK_SIZES = {
     "w2048": (_sutuvik(2048, "RMBMRMBM", 16, 2, 128, 64, 64, 128, 16, 4, 1376, 128), *ZISESUN_SIZES["w2048"][::-1]),
     "w4096": (_sutuvik(4096, "RMBM", 32, 8, 128, 128, 64, 128, 32, 4, 2048, 256), *ZISESUN_SIZES["w4096"][::-1]),
 }
-NEAREST_DESIGN = {"lazilorn": "zisesun", "bilipel": "lodalix", "sutuvik": "zisesun"}
+
+
+def _bozevik(width, layers, heads, dim, rot_dim, kv_rank, q_rank, ff, experts, top, expert_ff, vocab=32000) -> dict:
+    """``layers``: a string of D (latent attention on its own latent, a dense feed-forward) and S (on the latent of the
+    D layer before it, routed experts and a shared one of the same size)."""
+    sizes = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=dim, kv_rank=kv_rank, q_rank=q_rank,
+                 scale=(dim + rot_dim) ** -0.5, rot=dict(base=10000.0, dims=rot_dim))
+    unit = dict(ff=expert_ff, limit=7.0)
+    entries = []
+    for index, letter in enumerate(layers):
+        if letter == "D":
+            owner = index
+            entries.append(dict(type="latent_attention", mixer=sizes, mlp=dict(kind="dense", ff=ff, limit=7.0)))
+        else:
+            entries.append(dict(type="latent_attention", mixer=dict(sizes, kv_from=owner),
+                                mlp=dict(kind="moe", expert=unit, router=dict(experts=experts, top=top), shared=unit)))
+    return dict(architecture="Bozevik", vocab=vocab, width=width, logit_scale=0.25, norm=dict(eps=1e-6), layers=entries)
+
+
+# (Bozevik configuration, the Qwen2 dense shape of equal width, layers, heads and ACTIVE feed-forward size, and the
+# Lodalix configuration of that size: the design whose parts are nearest, latent attention with layers that read an
+# earlier layer's latent, and the same gated activation)
+BOZEVIK_SIZES = {
+    "w2048": (_bozevik(2048, "DSDSDSDS", 16, 128, 64, 512, 768, 5504, 16, 3, 1376), *LODALIX_SIZES["w2048"][::-1]),
+    "w4096": (_bozevik(4096, "DSDS", 32, 128, 64, 512, 1536, 8192, 32, 3, 2048), *LODALIX_SIZES["w4096"][::-1]),
+}
+NEAREST_DESIGN = {"lazilorn": "zisesun", "bilipel": "lodalix", "sutuvik": "zisesun", "bozevik": "lodalix"}
+DESIGNS = ("zisesun", "lodalix", "lazilorn", "bilipel", "sutuvik", "bozevik")
 
 
 def _time_step_function(cfg: dict, batch: int, steps: int, warmup: int, only: str = "all") -> dict:
@@ -786,7 +819,7 @@ def run_design(args: argparse.Namespace, design: str = "zisesun") -> int:
     import torch
 
     sizes = {"zisesun": ZISESUN_SIZES, "lodalix": LODALIX_SIZES, "lazilorn": LAZILORN_SIZES,
-             "bilipel": BILIPEL_SIZES, "sutuvik": SUTUVIK_SIZES}[design]
+             "bilipel": BILIPEL_SIZES, "sutuvik": SUTUVIK_SIZES, "bozevik": BOZEVIK_SIZES}[design]
     near = NEAREST_DESIGN.get(design)
     title = design.capitalize()
 
@@ -862,12 +895,12 @@ def main() -> int:
                              "default is 2048; longer ones are for profiles of long contexts, own arm only)")
     parser.add_argument("--impl", default="own", choices=("own", "reference"))
     parser.add_argument("--size", default="all", help="--config zisesun or lodalix: one of its sizes (w2048, w4096)")
-    parser.add_argument("--model", default="both", choices=("both", "zisesun", "lodalix", "lazilorn", "bilipel", "sutuvik", "qwen2"),
-                        help="--config zisesun, lodalix, lazilorn, bilipel or sutuvik: only that design, or only its dense peer "
-                             "(--config lazilorn or sutuvik --model zisesun, --config bilipel --model lodalix: only the nearest "
-                             "design's configuration of that size)")
+    parser.add_argument("--model", default="both", choices=("both", *DESIGNS, "qwen2"),
+                        help="--config with a design's name: only that design, or only its dense peer "
+                             "(--config lazilorn or sutuvik --model zisesun, --config bilipel or bozevik --model lodalix: only "
+                             "the nearest design's configuration of that size)")
     parser.add_argument("--config", default="3b",
-                        choices=("3b", "7b-mixed", "14b-pressure", "zisesun", "lodalix", "lazilorn", "bilipel", "sutuvik"),
+                        choices=("3b", "7b-mixed", "14b-pressure", *DESIGNS),
                         help="the benchmark configuration whose line is printed (default: the 3B line, "
                              "which also carries the other two as points)")
     parser.add_argument("--quick", action="store_true",
@@ -891,7 +924,7 @@ def main() -> int:
         CONTEXT = min(limit, PROMPT_TOKENS + max(2048, room))
     if args.impl == "reference":
         return run_reference(args)
-    if args.config in ("zisesun", "lodalix", "lazilorn", "bilipel", "sutuvik"):
+    if args.config in DESIGNS:
         return run_design(args, args.config)
     if args.config != "3b":
         return run_other_config(args)
