@@ -15,6 +15,8 @@ import os
 from ctypes import c_float, c_int, c_void_p
 from typing import Any
 
+import numpy as np
+
 from ..lazy import Accumulated, DepthUpdate, GateUpWeight, NormedInput, NormedUpdate, Partials, ResidualSink, StreamUpdate, WeightedTerms  # noqa: F401  (re-exported)
 from .build import load_library
 
@@ -37,6 +39,14 @@ STREAM_MAX_ROWS = 16
 # Up to this many rows a projection adds itself into the residual stream, or rotates and stores
 # q/k/v (cluster epilogues of the streaming kernel): every row count that kernel takes.
 FUSED_RESIDUAL_MAX_ROWS = STREAM_MAX_ROWS
+
+
+# Attention over a cached latent: portions of at least this many tokens in a step attend over keys and values expanded
+# from the latents (fewer: over the latents themselves), if they see at most so many keys together; the expanded rows
+# of as many heads as fit this many bytes are made at a time.
+LATENT_PROMPT_TOKENS = 48
+LATENT_PROMPT_KEYS = 1 << 17
+LATENT_PROMPT_BYTES = 1 << 28
 
 
 class _Lib:
@@ -1088,11 +1098,95 @@ class Ops:
                     "cie_latent_attention_tensor",
                     [v, v, i, i, v, v, v, v, v, v, v, i, i, v, f, i, i, v, i, i, i, i, i, f, i, i, i, i, v, v])
                 self._latent_tensor_supports = tensor.handle.cie_latent_attention_tensor_supports
+            self._latent_prompt_lib = None
+            if self.code == BF16 and os.environ.get("CIE_LATENT_PROMPT", "1") != "0":
+                prompt = _Lib(load_library("latent_prompt.cu"))
+                self._latent_gather = prompt.function("cie_latent_gather", [v, v, v, i, v, v, i, i, i, i, i, v, v, i, v, v])
+                self._latent_prompt = prompt.function(
+                    "cie_latent_prompt",
+                    [v, i, v, i, v, i, v, v, v, i, v, i, v, v, v, v, f, i, i, i, i, i, i, i, i, f, v, v])
+                self._latent_prompt_lib = prompt
 
     def require_latent(self) -> int:
         """Builds, at model set-up, the kernels of attention over a cached latent; returns the largest latent they take."""
         self._load_latent()
         return self.latent_max_rank
+
+    def expands_latents(self, dim: int, rot: int, vdim: int, rank: int) -> bool:
+        """Whether ``latent_prompt`` takes heads of these sizes."""
+        self._load_latent()
+        return self._latent_prompt_lib is not None and bool(
+            self._latent_prompt_lib.handle.cie_latent_prompt_supports(dim, rot, vdim, rank))
+
+    @staticmethod
+    def plan_latent_prompt(host: Any, window: int = 0) -> dict[str, Any]:
+        """Work lists of ``latent_prompt`` for a step's portions (empty: too few tokens for expanding their context to
+        pay, or too many keys): ``portions`` [count + 1, 3] = (request, first row, first key), closed by the number of
+        rows; ``block_portion``: the portion that every 128th row belongs to; ``tiles`` [tiles, 4] = (request, first
+        token in the portion, first row, first key), those with the most keys first."""
+        first = host.num_single
+        lens = host.query_lens[first:].astype(np.int64)
+        if lens.sum() < LATENT_PROMPT_TOKENS:
+            return {}
+        contexts = host.context_lens[first:].astype(np.int64)
+        first_key = np.maximum(contexts + 1 - window, 0) if window > 0 else np.zeros_like(contexts)
+        ends = np.cumsum(contexts + lens - first_key)
+        if ends[-1] > LATENT_PROMPT_KEYS:
+            return {}
+        starts = np.concatenate([[0], ends[:-1]])
+        requests = np.arange(first, first + len(lens))
+        portions = np.stack([np.append(requests, 0), np.append(starts, ends[-1]), np.append(first_key, 0)], axis=1)
+        block_portion = np.searchsorted(ends, np.arange(0, ends[-1], 128), side="right")
+        counts = -(-lens // 128)
+        owner = np.repeat(np.arange(len(lens)), counts)
+        q0 = 128 * (np.arange(len(owner)) - np.repeat(np.cumsum(counts) - counts, counts))
+        keys = contexts[owner] - first_key[owner] + np.minimum(q0 + 128, lens[owner])
+        tiles = np.stack([requests[owner], q0, starts[owner], first_key[owner]], axis=1)[np.argsort(-keys, kind="stable")]
+        return {name: np.ascontiguousarray(array, dtype=np.int32)
+                for name, array in (("portions", portions), ("block_portion", block_portion), ("tiles", tiles))}
+
+    def latent_prompt(self, q: Any, out: Any, ctx: Any, kv: Any, rotation: Any, plan: dict[str, Any], w_kv: Any, sink: Any,
+                      heads: int, dim: int, rot: int, vdim: int, rank: int, scale: float, window: int = 0,
+                      gate: Any = None) -> None:
+        """Attention of a step's portions (``plan``) with every head's keys and values expanded from the cached latents:
+        ``q`` float32 rows [heads * (dim + rot)], head by head plain part and rotated part (rotated here); ``w_kv``
+        [heads * (dim + vdim), rank], per head its key rows and then its value rows; ``out`` bfloat16 rows
+        [heads * vdim], times sigmoid(``gate``) if there is one.  Expanding happens for as many heads at a time as fit
+        a bounded buffer."""
+        self._flush()
+        self._load_latent()
+        torch = self.torch
+        blocks, tiles = plan["block_portion"], plan["tiles"]
+        rows, count = 128 * blocks.shape[0], plan["portions"].shape[0] - 1
+        table = ctx.block_tables[kv.group]
+        # no step's portions see more keys than the pages hold
+        most = max(rows, min(LATENT_PROMPT_KEYS, kv.num_pages * kv.page_size) // 128 * 128 + 128)
+
+        def buffer(tag: str, elements: int, reserve: int) -> Any:
+            return self.scratch(tag, (elements + 1) // 2, reserve=(reserve + 1) // 2).view(torch.bfloat16)[:elements]
+
+        c_rows = buffer(f"latent.c_rows.{rank}", rows * rank, most * rank).view(rows, rank)
+        r_rows = buffer(f"latent.r_rows.{rot}", rows * rot, most * rot).view(rows, rot)
+        self.launches += 1
+        self._latent_gather(_ptr(kv.k), _ptr(kv.v), _ptr(plan["portions"]), count, _ptr(blocks), _ptr(table),
+                            table.shape[1], kv.num_pages, kv.page_size, rank, rot, _ptr(c_rows), _ptr(r_rows), rows,
+                            _ptr(self.error_word), self.stream)
+        width = dim + vdim
+        limit = LATENT_PROMPT_BYTES // 2
+        at_once = max(1, min(heads, limit // (rows * width)))
+        expanded = buffer("latent.expanded", rows * at_once * width,
+                          max(most * width, min(limit, most * heads * width)))
+        for head0 in range(0, heads, at_once):
+            part = min(at_once, heads - head0)
+            kv_rows = expanded[: rows * part * width].view(rows, part * width)
+            self.linear(c_rows, w_kv[head0 * width:(head0 + part) * width], None, kv_rows)
+            self.launches += 1
+            self._latent_prompt(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(gate),
+                                gate.stride(0) if gate is not None else 0, _ptr(sink), _ptr(kv_rows), _ptr(r_rows), rows,
+                                _ptr(tiles), tiles.shape[0], _ptr(ctx.context_lens), _ptr(ctx.query_lens),
+                                _ptr(ctx.query_start), _ptr(rotation.inv_freq), float(rotation.magnitude),
+                                int(rotation.interleaved), int(rotation.dims), head0, part, dim, rot, vdim, int(window),
+                                float(scale), _ptr(self.error_word), self.stream)
 
     def latent_prepare(self, down: Any, q_out: Any, q_gain: Any, kv_gain: Any, ctx: Any, kv: Any, rotation: Any,
                        q_rank: int, rank: int, rot: int, eps: float, has_kv: bool, write_cache: bool) -> None:

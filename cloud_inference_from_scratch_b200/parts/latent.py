@@ -16,6 +16,10 @@ the latent space (``q' = W_uk[j]^T q_plain``: a product per head), attention run
 [c | key part] for all heads at once and sums latents, and ``W_uv[j]`` is applied to the sum (again a
 product per head, with the gate in its epilogue).  Scores, weights, norms and angles are float32.
 
+For the portions of prompts, when a step brings enough tokens of them (bfloat16, sizes the tensor-core kernel takes), it
+is the other way round: the keys and values of all heads are worked out once for everything the portions see (one
+product over the gathered latents) and attention runs over them, per head; no query is carried into the latent space.
+
 ``shares_cache``: the layer has no ``W_dkv`` and no latent norm of its own; it reads the rows another
 layer of equal ``kv_rank``, ``rot_dim`` and rotation wrote (the schedule's ``reads_cache_of``).
 
@@ -115,6 +119,11 @@ class LatentAttention(Mixer):
         self.w_absorb = ops.prepare_weight(tensors[n["uk"]]).view(heads, self.head_dim, self.kv_rank).contiguous()
         self.w_expand = (ops.prepare_weight(tensors[n["uv"]]).view(heads, self.value_dim, self.kv_rank)
                          .transpose(1, 2).contiguous())
+        self.w_kv = None
+        if ops.expands_latents(self.head_dim, self.rot_dim, self.value_dim, self.kv_rank):
+            self.w_kv = ops.prepare_weight(torch.cat(
+                [tensors[n["uk"]].view(heads, self.head_dim, self.kv_rank),
+                 tensors[n["uv"]].view(heads, self.value_dim, self.kv_rank)], dim=1).reshape(-1, self.kv_rank))
         self.w_o = ops.prepare_weight(tensors[n["o"]])
         self.q_gain = tensors[n["dq.norm"]].contiguous() if self.q_rank else None
         self.kv_gain = tensors[n["dkv.norm"]].contiguous() if not self.shares_cache else None
@@ -124,6 +133,14 @@ class LatentAttention(Mixer):
         self.rotation = SimpleNamespace(
             inv_freq=inv_freq.to(runtime.device).contiguous(), magnitude=self.position.magnitude,
             interleaved=self.position.pairing == "interleaved", dims=self.position.rotary_dim)
+
+    @property
+    def plan_key(self):
+        """Work lists of the expanded form of prompt portions; layers of one window share them."""
+        return ("latent_prompt", self.window) if getattr(self, "w_kv", None) is not None else None
+
+    def plan(self, host, cache):
+        return self.runtime.ops.plan_latent_prompt(host, self.window)
 
     def forward(self, x, ctx, binding):
         import torch
@@ -148,14 +165,22 @@ class LatentAttention(Mixer):
             if not self.shares_cache:
                 ops.latent_prepare(down[:, self.q_columns:], None, None, self.kv_gain, ctx, kv, self.rotation, 0,
                                    self.kv_rank, self.rot_dim, self.norm_eps, True, binding.owns_cache)
-        q_absorbed = rt.workspace.get("latent.q_absorbed", tokens, heads * self.kv_rank, f32)
-        ops.head_linear(q, self.q_head, self.w_absorb, q_absorbed, self.kv_rank, heads)
-        summed = rt.workspace.get("latent.sum", tokens, heads * self.kv_rank, f32)
-        ops.latent_attention(q_absorbed, q[:, self.head_dim:], self.q_head, summed, ctx, kv, self.rotation,
-                             self.sinks, heads, self.kv_rank, self.rot_dim, self.scale, window=self.window)
         mixed = rt.workspace.get("latent.out", tokens, self.out_width, rt.dtype)
-        ops.head_linear(summed, self.kv_rank, self.w_expand, mixed, self.value_dim, heads,
-                        gate=down[:, self.gate_column:] if self.gate else None)
+        gate = down[:, self.gate_column:] if self.gate else None
+        plan = (ctx.extras.get(self.plan_key) or None) if self.w_kv is not None else None
+        # with a plan only the leading rows, the step's single tokens, meet the latents themselves
+        few = ctx.num_single if plan else tokens
+        if few:
+            q_absorbed = rt.workspace.get("latent.q_absorbed", few, heads * self.kv_rank, f32)
+            ops.head_linear(q[:few], self.q_head, self.w_absorb, q_absorbed, self.kv_rank, heads)
+            summed = rt.workspace.get("latent.sum", few, heads * self.kv_rank, f32)
+            ops.latent_attention(q_absorbed, q[:few, self.head_dim:], self.q_head, summed, ctx, kv, self.rotation,
+                                 self.sinks, heads, self.kv_rank, self.rot_dim, self.scale, window=self.window)
+            ops.head_linear(summed, self.kv_rank, self.w_expand, mixed[:few], self.value_dim, heads,
+                            gate=gate[:few] if gate is not None else None)
+        if plan:
+            ops.latent_prompt(q, mixed, ctx, kv, self.rotation, plan, self.w_kv, self.sinks, heads, self.head_dim,
+                              self.rot_dim, self.value_dim, self.kv_rank, self.scale, window=self.window, gate=gate)
         update = rt.workspace.get("mixer.update32", tokens, self.hidden_size, f32)
         return ops.linear(mixed, self.w_o, None, update)
 
