@@ -33,34 +33,54 @@ __device__ __forceinline__ void pair_places(int i, int dims, int interleaved, in
 
 // ---------------------------------------------------------------- norms, rotation, cache write
 // down: float32 [T, stride]: [query latent (q_rank) | latent (rank) | key part (rot)]; the last two
-// only if has_kv.  q_out: [T, q_rank] in the compute dtype.
+// only if has_kv.  The row may still be `terms` partial sums of a product cut along K, `term_stride` elements apart.
+// q_out: [T, q_rank] in the compute dtype.
 template <typename T>
-__global__ void __launch_bounds__(128)
-latent_prepare_kernel(const float* __restrict__ down, int stride, T* __restrict__ q_out,
+__global__ void __launch_bounds__(256)
+latent_prepare_kernel(const float* __restrict__ down, int stride, int terms, size_t term_stride, T* __restrict__ q_out,
                       const float* __restrict__ q_gain, const float* __restrict__ kv_gain,
                       const int* __restrict__ positions, const int* __restrict__ request_of_token,
                       const int* __restrict__ table, int table_width, int num_pages, T* __restrict__ c_pool,
                       T* __restrict__ r_pool, const float* __restrict__ inv_freq, float magnitude, int interleaved,
                       int rot_dims, int q_rank, int rank, int rot, int page_size, float eps, int has_kv,
                       int write_cache, const int* __restrict__ active, int* err) {
-  __shared__ float scratch[33];
+  extern __shared__ __align__(16) float row_s[];        // the whole row, summed up
+  __shared__ float sums[2][32];
   pdl_wait();
   pdl_trigger();
-  const int t = blockIdx.x;
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float* row = down + (size_t)t * stride;
-  if (q_rank > 0) {
-    float sq = 0.f;
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) sq += row[i] * row[i];
-    const float inv = rsqrtf(block_sum(sq, scratch) / (float)q_rank + eps);
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
-      q_out[(size_t)t * q_rank + i] = from_float<T>(q_gain[i] * (row[i] * inv));
+  const bool keep = has_kv && write_cache && !(active && !active[request_of_token[t]]);   // not a row that only pads the batch
+  const int width = q_rank + (keep ? rank + rot : 0), latent_end = q_rank + rank;
+  float q_sq = 0.f, kv_sq = 0.f;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    float v = row[i];
+    for (int s = 1; s < terms; ++s) v += row[s * term_stride + i];
+    row_s[i] = v;
+    if (i < q_rank) q_sq = fmaf(v, v, q_sq);
+    else if (i < latent_end) kv_sq = fmaf(v, v, kv_sq);
   }
-  if (!has_kv || !write_cache) return;
-  if (active && !active[request_of_token[t]]) return;     // a row that only pads the batch
-  const float* kv = row + q_rank;
-  float sq = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) sq += kv[i] * kv[i];
-  const float inv = rsqrtf(block_sum(sq, scratch) / (float)rank + eps);
+  q_sq = warp_sum(q_sq);
+  kv_sq = warp_sum(kv_sq);
+  if (lane == 0) {
+    sums[0][warp] = q_sq;
+    sums[1][warp] = kv_sq;
+  }
+  __syncthreads();
+  q_sq = kv_sq = 0.f;
+  for (int w = 0; w < (int)blockDim.x / 32; ++w) {
+    q_sq += sums[0][w];
+    kv_sq += sums[1][w];
+  }
+  if (q_rank > 0) {
+    const float inv = rsqrtf(q_sq / (float)q_rank + eps);
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
+      q_out[(size_t)t * q_rank + i] = from_float<T>(q_gain[i] * (row_s[i] * inv));
+  }
+  if (!keep) return;
+  const float* kv = row_s + q_rank;
+  const float inv = rsqrtf(kv_sq / (float)rank + eps);
   const int pos = positions[t];
   const int page = table[(size_t)request_of_token[t] * table_width + pos / page_size];
   if (page < 0 || page >= num_pages) {
@@ -197,6 +217,70 @@ head_linear_few_kernel(const float* __restrict__ x, int x_stride, int x_head, co
   for (int e = threadIdx.x; e < tokens * kFewColumns; e += blockDim.x) {
     const int i = e / kFewColumns, c = e % kFewColumns;
     const int column = blockIdx.y * kFewColumns + c;
+    if (column >= N) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int sl = 0; sl < kFewSlices; ++sl) v += sums[sl][i][c];
+    if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)i * gate_stride + (size_t)h * N + column]));
+    out[(size_t)i * out_stride + (size_t)h * out_head + column] = from_float<TO>(v);
+  }
+}
+
+// The same with the block's weights [K][32] in shared memory, asked for before the kernel waits for the one before it
+// (nothing writes weights), and x as it lies: a slice takes every eighth group of four k.  bfloat16 weights with N a
+// multiple of 8, K a multiple of 4 that fits.
+template <typename TO, int TOKENS>
+__global__ void __launch_bounds__(kFewSlices * kFewColumns)
+head_linear_staged_kernel(const float* __restrict__ x, int x_stride, int x_head, const __nv_bfloat16* __restrict__ w,
+                          TO* __restrict__ out, int out_stride, int out_head, const float* __restrict__ gate,
+                          int gate_stride, int tokens, int K, int N) {
+  extern __shared__ __align__(16) float staged[];
+  float* xs = staged;                                                                       // [TOKENS][K]
+  __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(xs + (size_t)TOKENS * K);            // [K][32]
+  __shared__ float sums[kFewSlices][TOKENS][kFewColumns + 1];
+  const int h = blockIdx.x, column0 = blockIdx.y * kFewColumns;
+  const int slice = threadIdx.x / kFewColumns, lane = threadIdx.x % kFewColumns;
+  const __nv_bfloat16* wh = w + (size_t)h * K * N + column0;
+  const int pieces = min(4, (N - column0) / 8);
+  for (int e = threadIdx.x; e < K * 4; e += blockDim.x) {
+    const int k = e >> 2, p = e & 3;
+    const unsigned dst = (unsigned)__cvta_generic_to_shared(ws + k * kFewColumns + p * 8);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(wh + (p < pieces ? (size_t)k * N + p * 8 : 0)),
+                 "r"(p < pieces ? 16 : 0) : "memory");
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  pdl_wait();
+  pdl_trigger();
+  const int quads = K / 4;
+  for (int i = 0; i < TOKENS; ++i)
+    for (int k = threadIdx.x; k < quads; k += blockDim.x)
+      reinterpret_cast<float4*>(xs + (size_t)i * K)[k] =
+          i < tokens ? *reinterpret_cast<const float4*>(x + (size_t)i * x_stride + (size_t)h * x_head + 4 * k)
+                     : make_float4(0.f, 0.f, 0.f, 0.f);
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  float acc[TOKENS];
+#pragma unroll
+  for (int i = 0; i < TOKENS; ++i) acc[i] = 0.f;
+#pragma unroll 2
+  for (int k = slice; k < quads; k += kFewSlices) {
+    float wv[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) wv[u] = __bfloat162float(ws[(4 * k + u) * kFewColumns + lane]);
+#pragma unroll
+    for (int i = 0; i < TOKENS; ++i) {
+      const float4 v = reinterpret_cast<const float4*>(xs + (size_t)i * K)[k];
+      acc[i] = fmaf(v.x, wv[0], acc[i]);
+      acc[i] = fmaf(v.y, wv[1], acc[i]);
+      acc[i] = fmaf(v.z, wv[2], acc[i]);
+      acc[i] = fmaf(v.w, wv[3], acc[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < TOKENS; ++i) sums[slice][i][lane] = acc[i];
+  __syncthreads();
+  for (int e = threadIdx.x; e < tokens * kFewColumns; e += blockDim.x) {
+    const int i = e / kFewColumns, c = e % kFewColumns, column = column0 + c;
     if (column >= N) continue;
     float v = 0.f;
 #pragma unroll
@@ -389,29 +473,48 @@ latent_attention_kernel(const float* __restrict__ q_abs, const float* __restrict
   }
 }
 
-// Joins the key ranges of every (token, head): grid (tokens, heads), in ascending range order.
-__global__ void __launch_bounds__(128)
+// Joins the key ranges of every (token, head): grid (tokens, heads), in ascending range order.  The ranges' weights are
+// worked out side by side first; a thread's loads of a column's shares do not depend on one another.
+constexpr int kMergeThreads = 128;
+__global__ void __launch_bounds__(kMergeThreads)
 latent_merge_kernel(const float* __restrict__ part, float* __restrict__ out, const int* __restrict__ positions,
                     const float* __restrict__ sink, int heads, int rank, int range_keys, int ranges, int window) {
-  constexpr int kHeld = 256;          // weights of this many ranges are worked out once and kept
-  __shared__ float held[kHeld];
+  constexpr int kHeld = 1024;         // weights of this many ranges are kept; those of more are worked out again
+  __shared__ float held[kHeld], scratch[33], tops[kMergeThreads / 32];
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x, h = blockIdx.y;
   const int seen = window > 0 ? min(positions[t] + 1, window) : positions[t] + 1;      // visible keys
   const int used = min(ranges, (seen + range_keys - 1) / range_keys);
-  const float* share = part + ((size_t)t * heads + h) * ranges * (rank + 2);
-  float top = sink ? sink[h] : -FLT_MAX;
-  for (int r = 0; r < used; ++r) top = fmaxf(top, share[(size_t)r * (rank + 2)]);
-  for (int r = threadIdx.x; r < min(used, kHeld); r += blockDim.x) held[r] = expf(share[(size_t)r * (rank + 2)] - top);
+  const size_t stride = rank + 2;
+  const float* share = part + ((size_t)t * heads + h) * ranges * stride;
+  float top = -FLT_MAX;
+  for (int r = threadIdx.x; r < used; r += kMergeThreads) {
+    const float m = share[r * stride];
+    if (r < kHeld) held[r] = m;
+    top = fmaxf(top, m);
+  }
+  top = warp_max(top);
+  if ((threadIdx.x & 31) == 0) tops[threadIdx.x >> 5] = top;
   __syncthreads();
-  auto weight = [&](int r) { return r < kHeld ? held[r] : expf(share[(size_t)r * (rank + 2)] - top); };
-  float total = sink ? expf(sink[h] - top) : 0.f;
-  for (int r = 0; r < used; ++r) total += share[(size_t)r * (rank + 2) + 1] * weight(r);
+  top = sink ? sink[h] : -FLT_MAX;
+#pragma unroll
+  for (int w = 0; w < kMergeThreads / 32; ++w) top = fmaxf(top, tops[w]);
+  float total = 0.f;
+  for (int r = threadIdx.x; r < used; r += kMergeThreads) {
+    const float w = expf((r < kHeld ? held[r] : share[r * stride]) - top);
+    if (r < kHeld) held[r] = w;
+    total = fmaf(share[r * stride + 1], w, total);
+  }
+  total = block_sum(total, scratch);       // its barriers also publish the weights
+  if (sink) total += expf(sink[h] - top);
   const float inv = 1.f / total;
-  for (int col = threadIdx.x; col < rank; col += blockDim.x) {
+  for (int col = threadIdx.x; col < rank; col += kMergeThreads) {
+    const float* column = share + 2 + col;
     float a = 0.f;
-    for (int r = 0; r < used; ++r) a = fmaf(share[(size_t)r * (rank + 2) + 2 + col], weight(r), a);
+#pragma unroll 8
+    for (int r = 0; r < min(used, kHeld); ++r) a = fmaf(column[r * stride], held[r], a);
+    for (int r = kHeld; r < used; ++r) a = fmaf(column[r * stride], expf(share[r * stride] - top), a);
     out[((size_t)t * heads + h) * rank + col] = a * inv;
   }
 }
@@ -423,7 +526,7 @@ latent_merge_kernel(const float* __restrict__ part, float* __restrict__ out, con
   else if ((code) == cie::kBFloat16) { using T = __nv_bfloat16; __VA_ARGS__ } \
   else CIE_FAIL("%s: unknown dtype code %d", name, (code));
 
-extern "C" int cie_latent_prepare(const float* down, int stride, void* q_out, const float* q_gain,
+extern "C" int cie_latent_prepare(const float* down, int stride, int terms, long long term_stride, void* q_out, const float* q_gain,
                                   const float* kv_gain, const int* positions, const int* request_of_token,
                                   const int* table, int table_width, int num_pages, void* c_pool, void* r_pool,
                                   const float* inv_freq, float magnitude, int interleaved, int rot_dims,
@@ -433,9 +536,16 @@ extern "C" int cie_latent_prepare(const float* down, int stride, void* q_out, co
   using namespace cie;
   if (tokens <= 0) return 0;
   if (rot_dims % 2 || rot_dims > rot) CIE_FAIL("latent_prepare: %d rotated dims of %d", rot_dims, rot);
+  if (terms < 1 || terms > 64) CIE_FAIL("latent_prepare: 1..64 terms, got %d", terms);
+  const size_t smem = (size_t)(q_rank + (has_kv ? rank + rot : 0)) * sizeof(float);
+  if (smem > 200 * 1024) CIE_FAIL("latent_prepare: a row of %zu bytes does not fit shared memory", smem);
+  // few tokens: more threads a token hide the trips to memory; many: a block's reductions cost less with fewer
+  const int threads = tokens <= 148 ? 256 : 128;
   DISPATCH_DTYPE(dtype, "latent_prepare", {
-    CIE_LAUNCH("latent_prepare", latent_prepare_kernel<T>, dim3(tokens), dim3(128), 0, (cudaStream_t)stream, down,
-               stride, (T*)q_out, q_gain, kv_gain, positions, request_of_token, table, table_width, num_pages,
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(latent_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      CIE_FAIL("latent_prepare: cannot reserve %zu bytes of shared memory", smem);
+    CIE_LAUNCH("latent_prepare", latent_prepare_kernel<T>, dim3(tokens), dim3(threads), smem, (cudaStream_t)stream, down,
+               stride, terms, (size_t)term_stride, (T*)q_out, q_gain, kv_gain, positions, request_of_token, table, table_width, num_pages,
                (T*)c_pool, (T*)r_pool, inv_freq, magnitude, interleaved, rot_dims, q_rank, rank, rot, page_size,
                eps, has_kv, write_cache, active, err);
   })
@@ -451,6 +561,27 @@ extern "C" int cie_head_linear(const float* x, int x_stride, int x_head, const v
   const dim3 grid = few ? dim3(heads, (N + kFewColumns - 1) / kFewColumns)
                         : dim3((tokens + kHeadTokens - 1) / kHeadTokens, heads, (N + kHeadColumns - 1) / kHeadColumns);
   if (grid.y > 65535 || grid.z > 65535) CIE_FAIL("head_linear: too many heads or columns");
+  const int staged_tokens = tokens <= 8 ? 8 : kHeadTokens;
+  const size_t staged = (size_t)K * (staged_tokens * sizeof(float) + kFewColumns * sizeof(__nv_bfloat16));
+  if (few && w_dtype == kBFloat16 && K % 4 == 0 && N % 8 == 0 && x_stride % 4 == 0 && x_head % 4 == 0 && staged <= 160 * 1024 &&
+      ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0) {
+#define CIE_HEAD_STAGED(TO, TOKENS)                                                                                       \
+  do {                                                                                                                    \
+    static bool raised = false;                                                                                           \
+    if (!raised && cudaFuncSetAttribute(head_linear_staged_kernel<TO, TOKENS>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                        160 * 1024) != cudaSuccess)                                                       \
+      CIE_FAIL("head_linear: cannot raise the shared memory limit");                                                      \
+    raised = true;                                                                                                        \
+    CIE_LAUNCH("head_linear", (head_linear_staged_kernel<TO, TOKENS>), grid, dim3(kFewSlices * kFewColumns), staged,      \
+               (cudaStream_t)stream, x, x_stride, x_head, (const __nv_bfloat16*)w, (TO*)out, out_stride, out_head, gate,  \
+               gate_stride, tokens, K, N);                                                                                \
+  } while (0)
+    if (out_dtype == kFloat32) { if (staged_tokens == 8) CIE_HEAD_STAGED(float, 8); else CIE_HEAD_STAGED(float, kHeadTokens); }
+    else if (out_dtype == kBFloat16) { if (staged_tokens == 8) CIE_HEAD_STAGED(__nv_bfloat16, 8); else CIE_HEAD_STAGED(__nv_bfloat16, kHeadTokens); }
+    else CIE_FAIL("head_linear: output dtype %d", out_dtype);
+#undef CIE_HEAD_STAGED
+    return 0;
+  }
 #define CIE_HEAD_LINEAR(TW, TO)                                                                                   \
   if (few) {                                                                                                      \
     CIE_LAUNCH("head_linear", (head_linear_few_kernel<TW, TO>), grid, dim3(kFewSlices * kFewColumns), 0,          \
@@ -495,7 +626,7 @@ extern "C" int cie_latent_merge(const float* part, float* out, const int* positi
                                 int heads, int rank, int range_keys, int ranges, int window, void* stream) {
   using namespace cie;
   if (tokens <= 0) return 0;
-  CIE_LAUNCH("latent_merge", latent_merge_kernel, dim3(tokens, heads), dim3(128), 0, (cudaStream_t)stream, part, out,
+  CIE_LAUNCH("latent_merge", latent_merge_kernel, dim3(tokens, heads), dim3(kMergeThreads), 0, (cudaStream_t)stream, part, out,
              positions, sink, heads, rank, range_keys, ranges, window);
   return 0;
 }
@@ -532,7 +663,7 @@ extern "C" int cie_latent_attention(const float* q_abs, const float* q_raw, int 
                heads, rank, rot, page_size, scale, range_keys, ranges, window, err);
   })
   if (ranges > 1)
-    CIE_LAUNCH("latent_merge", latent_merge_kernel, dim3(tokens, heads), dim3(128), 0, (cudaStream_t)stream, part, out,
+    CIE_LAUNCH("latent_merge", latent_merge_kernel, dim3(tokens, heads), dim3(kMergeThreads), 0, (cudaStream_t)stream, part, out,
                positions, sink, heads, rank, range_keys, ranges, window);
   return 0;
 }

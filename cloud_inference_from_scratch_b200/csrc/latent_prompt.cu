@@ -7,6 +7,8 @@
 //
 //   latent_gather     the cached rows a step's portions can see, request after request, out of the pages: latents
 //                     [keys][rank] and rotated key parts [keys][rot]
+//   latent_queries    the queries, float32, rounded to bfloat16 once, their rotated part after the rotation; every part of
+//                     a head padded with zeros to whole steps of 16
 //   latent_prompt     softmax attention of 128 tokens of one request and one head a CTA over its expanded rows
 //
 // In a CTA of latent_prompt keys go by in tiles of 128:
@@ -19,9 +21,8 @@
 //                     as TWO bfloat16 terms (the weight rounded, and what the rounding left), both multiplied with V
 //                     from there.  Maxima, sums and denominators are float32.  At the end the groups' halves join.
 //
-// The query comes as float32 and is rounded to bfloat16 once, its rotated part after the rotation.  Options: a window,
-// a sink term in the denominator, a gate on the result.  Every wait on an mbarrier is bounded.  A row's result depends
-// on its own request's rows alone.
+// Options: a window, a sink term in the denominator, a gate on the result.  Every wait on an mbarrier is bounded.  A
+// row's result depends on its own request's rows alone.
 #include "blackwell.cuh"
 #include "common.cuh"
 
@@ -90,10 +91,66 @@ latent_gather_kernel(const bf16* __restrict__ c_pool, const bf16* __restrict__ r
   for (int i = lane; i < rot / 8; i += 32) r_dst[i] = r_src ? r_src[i] : zero;
 }
 
+// ---------------------------------------------------------------- queries
+__host__ __device__ __forceinline__ int padded16(int columns) { return (columns + 15) / 16 * 16; }
+
+// A block per token: q [heads * (dim + rot)] float32 -> out [heads * (padded dim + padded rot)], 8 elements a thread at a time.
+constexpr int kMaxPairs = 128;
+__global__ void __launch_bounds__(256)
+latent_queries_kernel(const float* __restrict__ q, int q_stride, bf16* __restrict__ out, const int* __restrict__ positions,
+                      const float* __restrict__ inv_freq, float magnitude, int interleaved, int rot_dims, int heads, int dim,
+                      int rot) {
+  __shared__ float sin_s[kMaxPairs], cos_s[kMaxPairs];
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x, half = rot_dims / 2, plain = padded16(dim), width = plain + padded16(rot);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf((float)positions[t] * inv_freq[i], &s, &c);
+    sin_s[i] = s * magnitude;
+    cos_s[i] = c * magnitude;
+  }
+  __syncthreads();
+  const float* row = q + (size_t)t * q_stride;
+  uint4* dst = reinterpret_cast<uint4*>(out + (size_t)t * heads * width);
+  const int per_head = width / 8;
+  for (int piece = threadIdx.x; piece < heads * per_head; piece += blockDim.x) {
+    const int h = piece / per_head, column = (piece - h * per_head) * 8;
+    const float* src = row + (size_t)h * (dim + rot) + (column < plain ? column : dim + column - plain);
+    float v[8] = {};
+    const int first = column - plain;                       // in the rotated part
+    if (first < 0 ? column < dim : first < rot) {           // dim and rot are multiples of 8
+      const float4 lo = reinterpret_cast<const float4*>(src)[0], hi = reinterpret_cast<const float4*>(src)[1];
+      v[0] = lo.x; v[1] = lo.y; v[2] = lo.z; v[3] = lo.w;
+      v[4] = hi.x; v[5] = hi.y; v[6] = hi.z; v[7] = hi.w;
+      if (first >= 0) {
+        if (interleaved) {
+#pragma unroll
+          for (int e = 0; e < 8; e += 2) {
+            if (first + e >= rot_dims) continue;
+            const float u = v[e], w = v[e + 1], s = sin_s[(first + e) / 2], c = cos_s[(first + e) / 2];
+            v[e] = u * c - w * s;
+            v[e + 1] = w * c + u * s;
+          }
+        } else {
+          const float* part = row + (size_t)h * (dim + rot) + dim;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const int d = first + e;
+            if (d >= rot_dims) continue;
+            const int i = d < half ? d : d - half;
+            const float other = part[d < half ? d + half : d - half];
+            v[e] = d < half ? v[e] * cos_s[i] - other * sin_s[i] : v[e] * cos_s[i] + other * sin_s[i];
+          }
+        }
+      }
+    }
+    dst[piece] = make_uint4(pack(v[0], v[1]), pack(v[2], v[3]), pack(v[4], v[5]), pack(v[6], v[7]));
+  }
+}
+
 // ---------------------------------------------------------------- attention
 struct PromptArgs {
-  const float* q;            // token t, head h at q[t * q_stride + h * (dim + rot)]: [dim plain | rot not yet rotated]
-  int q_stride;
   bf16* out;                 // token t, head h at out[t * out_stride + h * vdim]
   int out_stride;
   const float* gate;         // like out (gate_stride), or nullptr
@@ -103,9 +160,7 @@ struct PromptArgs {
   const int* context_lens;
   const int* query_lens;
   const int* query_start;
-  const float* inv_freq;
-  float magnitude;
-  int interleaved, rot_dims;
+  int token0;                // the token that row 0 of the queries belongs to
   int head0;                 // first head of this launch (its columns of the expanded rows start at 0)
   int dim, rot, vdim;
   int window;
@@ -116,7 +171,8 @@ struct PromptArgs {
 __host__ __device__ __forceinline__ int pieces_of(int columns) { return (columns + PIECE - 1) / PIECE; }
 
 __global__ void __launch_bounds__(THREADS, 1)
-latent_prompt_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_constant__ CUtensorMap r_map, const PromptArgs a) {
+latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map,
+                     const __grid_constant__ CUtensorMap r_map, const PromptArgs a) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   const int k_plain = pieces_of(a.dim), k_pieces = k_plain + pieces_of(a.rot), v_pieces = pieces_of(a.vdim);
@@ -125,7 +181,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_co
   unsigned char* k_s = q_s + k_bytes;                  // [STAGES][k_bytes]
   unsigned char* v_s = k_s + STAGES * k_bytes;         // [STAGES][v_bytes]
   __shared__ __align__(8) uint64_t k_full[STAGES], k_empty[STAGES], v_full[STAGES], v_empty[STAGES];
-  __shared__ __align__(8) uint64_t s_full[2], p_full[2], pv_done[2];
+  __shared__ __align__(8) uint64_t q_full, s_full[2], p_full[2], pv_done[2];
   __shared__ uint32_t tmem_slot;
   __shared__ float m_s[2][BM], l_s[2][BM];
 
@@ -136,6 +192,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_co
       mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1);
       mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1);
     }
+    mbar_init(&q_full, 1);
     for (int g = 0; g < 2; ++g) { mbar_init(&s_full[g], 1); mbar_init(&p_full[g], BM); mbar_init(&pv_done[g], 1); }
     mbar_init_fence();
   }
@@ -152,50 +209,6 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_co
   const int tile0 = lowest / BN, tiles = (valid_hi + BN - 1) / BN - tile0;
 
   if (warp == MMA_WARP) tmem_alloc<TMEM_COLS>(&tmem_slot);
-  // the query rows, swizzled by hand: plain part, then rotated part, each in 64-column pieces, zeros beyond its size
-  for (int idx = tid; idx < BM * k_plain * 8; idx += THREADS) {
-    const int r = idx / (k_plain * 8), c = idx % (k_plain * 8);
-    uint4 value = make_uint4(0u, 0u, 0u, 0u);
-    if (r < ntok && c * 8 < a.dim) {           // dim is a multiple of 8
-      const float4* src = reinterpret_cast<const float4*>(a.q + (size_t)(first_token + r) * a.q_stride +
-                                                          (size_t)head * (a.dim + a.rot) + c * 8);
-      const float4 lo = src[0], hi = src[1];
-      value = make_uint4(pack(lo.x, lo.y), pack(lo.z, lo.w), pack(hi.x, hi.y), pack(hi.z, hi.w));
-    }
-    *reinterpret_cast<uint4*>(q_s + (c >> 3) * PIECE_BYTES + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = value;
-  }
-  {
-    unsigned char* rot_s = q_s + k_plain * PIECE_BYTES;
-    const int width = (k_pieces - k_plain) * PIECE, half = a.rot_dims / 2;
-    auto place = [&](int r, int d) {
-      return reinterpret_cast<bf16*>(rot_s + (d >> 6) * PIECE_BYTES + r * 128 + ((((d & 63) >> 3) ^ (r & 7)) << 4)) + (d & 7);
-    };
-    for (int idx = tid; idx < BM * half; idx += THREADS) {
-      const int r = idx / half, i = idx % half;
-      const int x = a.interleaved ? 2 * i : i, y = a.interleaved ? 2 * i + 1 : i + half;
-      float turned_x = 0.f, turned_y = 0.f;
-      if (r < ntok) {
-        const float* src = a.q + (size_t)(first_token + r) * a.q_stride + (size_t)head * (a.dim + a.rot) + a.dim;
-        float s, c;
-        sincosf((float)(key0 + pos_lo + r) * a.inv_freq[i], &s, &c);
-        s *= a.magnitude;
-        c *= a.magnitude;
-        const float u = src[x], v = src[y];
-        turned_x = u * c - v * s;
-        turned_y = v * c + u * s;
-      }
-      *place(r, x) = __float2bfloat16_rn(turned_x);
-      *place(r, y) = __float2bfloat16_rn(turned_y);
-    }
-    const int rest = width - a.rot_dims;
-    for (int idx = tid; idx < BM * rest; idx += THREADS) {
-      const int r = idx / rest, d = a.rot_dims + idx % rest;
-      float v = 0.f;
-      if (r < ntok && d < a.rot) v = a.q[(size_t)(first_token + r) * a.q_stride + (size_t)head * (a.dim + a.rot) + a.dim + d];
-      *place(r, d) = __float2bfloat16_rn(v);
-    }
-  }
-  fence_async_smem();
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -205,6 +218,13 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_co
   if (warp == TMA_WARP) {
     if (lane == 0) {
       const int column = blockIdx.y * (a.dim + a.vdim);
+      // the queries: plain part and rotated part begin at pieces of their own; what a piece holds beyond a part's padded
+      // columns takes part in no product
+      const int q_column = head * (padded16(a.dim) + padded16(a.rot)), q_row = first_token - a.token0;
+      mbar_expect_tx(&q_full, (uint32_t)k_bytes);
+      for (int p = 0; p < k_pieces; ++p)
+        tma_load_2d(q_s + p * PIECE_BYTES, &q_map, &q_full,
+                    q_column + (p < k_plain ? p * PIECE : padded16(a.dim) + (p - k_plain) * PIECE), q_row);
       for (int j = 0; j < tiles; ++j) {
         const int s = j % STAGES, row = row0 + (tile0 + j) * BN;
         const uint32_t before = ((j / STAGES) - 1) & 1;
@@ -246,6 +266,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_co
         tc_commit(&pv_done[g]);
         return true;
       };
+      alive = mbar_wait(&q_full, 0, a.err);
       for (int j = 0; j < tiles && alive; ++j) {
         const int g = j & 1, s = j % STAGES;
         // the weights of tile j - 2, which lie in this buffer, have been used
@@ -427,22 +448,37 @@ extern "C" int cie_latent_gather(const void* c_pool, const void* r_pool, const i
   return 0;
 }
 
-// kv_rows: [rows][heads * (dim + vdim)], per head its keys and then its values, for heads head0 .. head0 + heads - 1;
+// q: float32, token t, head h at q[t * q_stride + h * (dim + rot)]: [dim plain | rot not yet rotated]; out: [tokens][heads *
+// (dim padded to 16 + rot padded to 16)].
+extern "C" int cie_latent_queries(const float* q, int q_stride, void* out, const int* positions, const float* inv_freq,
+                                  float magnitude, int interleaved, int rot_dims, int tokens, int heads, int dim, int rot,
+                                  void* stream) {
+  if (tokens <= 0) return 0;
+  if (dim % 8 || rot % 8 || q_stride % 4 || ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out)) & 15))
+    CIE_FAIL("latent_queries: rows of heads of %d + %d elements must be 16-byte aligned", dim, rot);
+  if (rot_dims % 2 || rot_dims > rot || rot_dims / 2 > kMaxPairs) CIE_FAIL("latent_queries: %d rotated dims of %d", rot_dims, rot);
+  CIE_LAUNCH("latent_queries", latent_queries_kernel, dim3(tokens), dim3(256), 0, (cudaStream_t)stream, q, q_stride, (bf16*)out,
+             positions, inv_freq, magnitude, interleaved, rot_dims, heads, dim, rot);
+  return 0;
+}
+
+// queries: what latent_queries made of the tokens from token0 on (`tokens` rows, all_heads heads); kv_rows: [rows][heads *
+// (dim + vdim)], per head its keys and then its values, for heads head0 .. head0 + heads - 1;
 // r_rows: [rows][rot]; rows a multiple of 128.  tiles: [count][4] (see PromptArgs).
-extern "C" int cie_latent_prompt(const float* q, int q_stride, void* out, int out_stride, const float* gate, int gate_stride,
+extern "C" int cie_latent_prompt(const void* queries, int tokens, int all_heads, int token0, void* out, int out_stride, const float* gate, int gate_stride,
                                  const float* sink, const void* kv_rows, const void* r_rows, int rows, const int* tiles,
                                  int count, const int* context_lens, const int* query_lens, const int* query_start,
-                                 const float* inv_freq, float magnitude, int interleaved, int rot_dims, int head0, int heads,
-                                 int dim, int rot, int vdim, int window, float scale, int* err, void* stream) {
+                                 int head0, int heads, int dim, int rot, int vdim, int window, float scale, int* err, void* stream) {
   if (count <= 0 || heads <= 0) return 0;
   if (!cie_latent_prompt_supports(dim, rot, vdim, 8)) CIE_FAIL("latent_prompt: sizes %d + %d, %d", dim, rot, vdim);
-  if (rot_dims % 2 || rot_dims > rot) CIE_FAIL("latent_prompt: %d rotated dims of %d", rot_dims, rot);
-  if (q_stride % 4 || (reinterpret_cast<uintptr_t>(q) & 15)) CIE_FAIL("latent_prompt: query rows must be 16-byte aligned");
+  if (head0 < 0 || head0 + heads > all_heads) CIE_FAIL("latent_prompt: heads %d.. of %d", head0, all_heads);
   if (rows % 128 || out_stride % 8 || heads > 65535) CIE_FAIL("latent_prompt: %d rows, stride %d, %d heads", rows, out_stride, heads);
-  if ((reinterpret_cast<uintptr_t>(kv_rows) | reinterpret_cast<uintptr_t>(r_rows) | reinterpret_cast<uintptr_t>(out)) & 15)
+  if ((reinterpret_cast<uintptr_t>(kv_rows) | reinterpret_cast<uintptr_t>(r_rows) | reinterpret_cast<uintptr_t>(out) |
+       reinterpret_cast<uintptr_t>(queries)) & 15)
     CIE_FAIL("latent_prompt: operands must be 16-byte aligned");
-  CUtensorMap kv_map, r_map;
-  if (!tensor_map_bf16(kv_rows, rows, (long long)heads * (dim + vdim), BN, &kv_map) ||
+  CUtensorMap q_map, kv_map, r_map;
+  if (!tensor_map_bf16(queries, tokens, (long long)all_heads * (padded16(dim) + padded16(rot)), BM, &q_map) ||
+      !tensor_map_bf16(kv_rows, rows, (long long)heads * (dim + vdim), BN, &kv_map) ||
       !tensor_map_bf16(r_rows, rows, rot, BN, &r_map))
     CIE_FAIL("latent_prompt: cuTensorMapEncodeTiled failed");
   const size_t smem = prompt_smem(dim, rot, vdim);
@@ -452,8 +488,9 @@ extern "C" int cie_latent_prompt(const float* q, int q_stride, void* out, int ou
       CIE_FAIL("latent_prompt: cannot raise the shared memory limit");
     raised = true;
   }
-  const PromptArgs a{q, q_stride, (bf16*)out, out_stride, gate, gate_stride, sink, tiles, context_lens, query_lens, query_start,
-                     inv_freq, magnitude, interleaved, rot_dims, head0, dim, rot, vdim, window, scale * kLog2e, err};
-  CIE_LAUNCH("latent_prompt", latent_prompt_kernel, dim3(count, heads), dim3(THREADS), smem, (cudaStream_t)stream, kv_map, r_map, a);
+  const PromptArgs a{(bf16*)out, out_stride, gate, gate_stride, sink, tiles, context_lens, query_lens, query_start,
+                     token0, head0, dim, rot, vdim, window, scale * kLog2e, err};
+  CIE_LAUNCH("latent_prompt", latent_prompt_kernel, dim3(count, heads), dim3(THREADS), smem, (cudaStream_t)stream, q_map,
+             kv_map, r_map, a);
   return 0;
 }

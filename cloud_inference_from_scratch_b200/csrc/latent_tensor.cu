@@ -157,46 +157,6 @@ latent_attention_tensor_kernel(const float* __restrict__ q_abs, const float* __r
     const int* pages = table + (size_t)request_of_token[token[0]] * table_width;
 
     __syncthreads();      // a pass before this one is done with everything
-    // what no copy writes starts as zero (padding must not hold NaN patterns): the query rows, the weights,
-    // and the columns of every key row beyond [rank + rot]; rows past the last key are zero-filled by the copies
-    {
-      const int pad = ld - D;
-      for (int e = tid; e < ROWS * ld; e += blockDim.x) qs[e] = __float2bfloat16_rn(0.f);
-      for (int e = tid; e < 2 * kTile * pad; e += blockDim.x) ks[(e / pad) * ld + D + e % pad] = __float2bfloat16_rn(0.f);
-      for (int e = tid; e < 2 * ROWS * PLD; e += blockDim.x) ps[e] = __float2bfloat16_rn(0.f);
-    }
-    __syncthreads();
-
-    // the query rows: the latent part as it comes, the rotated part rotated here, both rounded once
-#pragma unroll
-    for (int tile = 0; tile < RT; ++tile) {
-      const int t = token[tile];
-      if (t < 0) continue;
-      bf16* rows = qs + tile * kRows * ld;
-      for (int e = tid; e < kRows * rank; e += blockDim.x) {
-        const int r = e / rank, d = e % rank;
-        if (h0 + r < heads) rows[r * ld + d] = __float2bfloat16_rn(q_abs[((size_t)t * heads + h0 + r) * rank + d]);
-      }
-      for (int e = tid; e < kRows * (rot_dims / 2); e += blockDim.x) {
-        const int r = e / (rot_dims / 2), i = e % (rot_dims / 2);
-        if (h0 + r >= heads) continue;
-        const float* qr = q_raw + (size_t)t * q_raw_stride + (size_t)(h0 + r) * q_raw_head;
-        const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + rot_dims / 2;
-        float sn, cs;
-        sincosf((float)position[tile] * inv_freq[i], &sn, &cs);
-        sn *= magnitude;
-        cs *= magnitude;
-        const float u = qr[a], v = qr[b];
-        rows[r * ld + rank + a] = __float2bfloat16_rn(u * cs - v * sn);
-        rows[r * ld + rank + b] = __float2bfloat16_rn(v * cs + u * sn);
-      }
-      for (int e = tid; e < kRows * (rot - rot_dims); e += blockDim.x) {
-        const int r = e / (rot - rot_dims), i = rot_dims + e % (rot - rot_dims);
-        if (h0 + r < heads)
-          rows[r * ld + rank + i] = __float2bfloat16_rn(q_raw[(size_t)t * q_raw_stride + (size_t)(h0 + r) * q_raw_head + i]);
-      }
-    }
-
     auto fetch = [&](int base, int buf) {
       // which row of the pools every key of the tile lives in
       if (tid < kTile) {
@@ -229,6 +189,60 @@ latent_attention_tensor_kernel(const float* __restrict__ q_abs, const float* __r
       cp_async_commit();
     };
 
+    // the first keys are on their way while the query rows are made
+    const int tiles = (end - begin + kTile - 1) / kTile;
+    fetch(begin, 0);
+    __syncthreads();
+    copy(0);
+    // the columns of the key rows that no copy writes start as zero (padding must not hold NaN patterns); rows past the
+    // last key are zero-filled by the copies
+    {
+      const int pad = ld - D;
+      for (int e = tid; e < 2 * kTile * pad; e += blockDim.x) ks[(e / pad) * ld + D + e % pad] = __float2bfloat16_rn(0.f);
+    }
+    // the query rows: the latent part as it comes, the rotated part rotated here, both rounded once; zeros for heads
+    // beyond the last, for an idle tile and up to the padded depth
+#pragma unroll
+    for (int tile = 0; tile < RT; ++tile) {
+      const int t = token[tile];
+      bf16* rows = qs + tile * kRows * ld;
+      const int quads = rank / 4;      // rank is a multiple of 8
+      const int row_step = kWarps * 32 / 16, r = tid / row_step;        // 16 threads a row
+      const bool real = t >= 0 && h0 + r < heads;
+      const float4* qa = reinterpret_cast<const float4*>(q_abs + ((size_t)(real ? t : 0) * heads + (real ? h0 + r : 0)) * rank);
+#pragma unroll 4
+      for (int c = tid % row_step; c < quads; c += row_step) {
+        const float4 v = real ? qa[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        *reinterpret_cast<__nv_bfloat162*>(rows + r * ld + 4 * c) = lo;
+        *reinterpret_cast<__nv_bfloat162*>(rows + r * ld + 4 * c + 2) = hi;
+      }
+      for (int e = tid; e < kRows * (rot_dims / 2); e += blockDim.x) {
+        const int q_row = e / (rot_dims / 2), i = e % (rot_dims / 2);
+        const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + rot_dims / 2;
+        float x = 0.f, y = 0.f;
+        if (t >= 0 && h0 + q_row < heads) {
+          const float* qr = q_raw + (size_t)t * q_raw_stride + (size_t)(h0 + q_row) * q_raw_head;
+          float sn, cs;
+          sincosf((float)position[tile] * inv_freq[i], &sn, &cs);
+          sn *= magnitude;
+          cs *= magnitude;
+          const float u = qr[a], v = qr[b];
+          x = u * cs - v * sn;
+          y = v * cs + u * sn;
+        }
+        rows[q_row * ld + rank + a] = __float2bfloat16_rn(x);
+        rows[q_row * ld + rank + b] = __float2bfloat16_rn(y);
+      }
+      const int rest = lay.depth - rank - rot_dims;
+      for (int e = tid; e < kRows * rest; e += blockDim.x) {
+        const int q_row = e / rest, i = rot_dims + e % rest;
+        float v = 0.f;
+        if (t >= 0 && h0 + q_row < heads && i < rot) v = q_raw[(size_t)t * q_raw_stride + (size_t)(h0 + q_row) * q_raw_head + i];
+        rows[q_row * ld + rank + i] = __float2bfloat16_rn(v);
+      }
+    }
+
     float o[RT][NT][4];
     float top[RT][2], sum[RT][2];     // running maxima of rows g and g + 8 of each tile (the same in every warp),
                                       // and this thread's share of the rows' sums (its own keys only)
@@ -240,10 +254,6 @@ latent_attention_tensor_kernel(const float* __restrict__ q_abs, const float* __r
       sum[tile][0] = sum[tile][1] = 0.f;
     }
 
-    const int tiles = (end - begin + kTile - 1) / kTile;
-    fetch(begin, 0);
-    __syncthreads();
-    copy(0);
     for (int i = 0; i < tiles; ++i) {
       const int buf = i & 1;
       const int base = begin + i * kTile;

@@ -52,7 +52,9 @@ struct Pending {
   int count;
   size_t stride, row_stride;
   const float* weights;    // not null: term s of row t is multiplied by weights[t * count + s]
-  const float* extra;      // not null: one more term, row t at t * hidden
+  const float* extra;      // not null: `extras` more terms (a result, whole or cut), term s of row t at t * hidden + s * extra_stride
+  int extras;
+  size_t extra_stride;
   const float* gain;       // [hidden], for kRms and kCentred
   float eps;
   int kind;
@@ -123,6 +125,7 @@ advance_kernel(Pending pending, Depth depth, T* __restrict__ out, const int* __r
     for (int p = 0; p < P; ++p)
 #pragma unroll
       for (int e = 0; e < V; ++e) y[p][e] = 0.f;
+#pragma unroll 4
     for (int s = 0; s < pending.count; ++s) {
       const float w = weights ? weights[s] : 1.f;
 #pragma unroll
@@ -139,10 +142,12 @@ advance_kernel(Pending pending, Depth depth, T* __restrict__ out, const int* __r
 #pragma unroll
       for (int p = 0; p < P; ++p) {
         if (!in(p)) continue;
-        float more[V];
-        load_v<V>(more, extra + p * step);
+        for (int s = 0; s < pending.extras; ++s) {
+          float more[V];
+          load_v<V>(more, extra + s * pending.extra_stride + p * step);
 #pragma unroll
-        for (int e = 0; e < V; ++e) y[p][e] += more[e];
+          for (int e = 0; e < V; ++e) y[p][e] += more[e];
+        }
       }
     }
     if (pending.kind == kPlain) {
@@ -311,7 +316,7 @@ extern "C" int cie_stream_step_max_width() { return 16 * 1024; }
 // asked for.
 extern "C" int cie_stream_advance(const float* base, long long base_stride, const float* terms, int count,
                                   long long stride, long long row_stride, const float* weights, const float* extra,
-                                  const float* gain, float eps, int pending_kind, const float* history,
+                                  int extras, long long extra_stride, const float* gain, float eps, int pending_kind, const float* history,
                                   long long history_stride, int states, const float* share, float* keep,
                                   long long keep_stride, float* stream, void* out, int out_kind, const int* rows,
                                   int out_rows, int hidden, const float* shift_share, float* state, long long state_stride,
@@ -321,16 +326,17 @@ extern "C" int cie_stream_advance(const float* base, long long base_stride, cons
   if (out_rows <= 0) return 0;
   if (hidden < 1 || hidden > cie_stream_step_max_width()) CIE_FAIL("stream_advance: a row of %d elements (at most %d)", hidden, cie_stream_step_max_width());
   if (terms && (count < 1 || count > kMaxTerms)) CIE_FAIL("stream_advance: 1..%d float32 terms, got %d", kMaxTerms, count);
+  if (extra && (extras < 1 || extras > kMaxTerms)) CIE_FAIL("stream_advance: 1..%d further terms, got %d", kMaxTerms, extras);
   if (pending_kind < 0 || pending_kind > 2 || out_kind < 0 || out_kind > 2) CIE_FAIL("stream_advance: kinds %d, %d", pending_kind, out_kind);
   if (terms && pending_kind != kPlain && !gain) CIE_FAIL("stream_advance: a normalised update needs its gain");
   if (rows && (keep || stream || out_kind == kShift)) CIE_FAIL("stream_advance: chosen rows are only read");
   if (out_kind == kShift && (!shift_share || !state)) CIE_FAIL("stream_advance: a shift needs its vector and state");
   if (out_kind == kShift && !singles && !stream && base_stride != hidden) CIE_FAIL("stream_advance: portions are shifted from the stream");
   if (out_kind == kNormed && !out_gain) CIE_FAIL("stream_advance: a norm needs its gain");
-  const Pending pending{terms, count, (size_t)stride, (size_t)row_stride, weights, extra, gain, eps, pending_kind};
+  const Pending pending{terms, count, (size_t)stride, (size_t)row_stride, weights, extra, extras, (size_t)extra_stride, gain, eps, pending_kind};
   const Depth depth{base, (size_t)base_stride, history, (size_t)history_stride, states, share, keep, (size_t)keep_stride, stream};
   const Shift shift{shift_share, state, state_stride, query_start, request_of_token, slots, active, max_slots};
-  const bool wide = hidden % 4 == 0 && base_stride % 4 == 0 && stride % 4 == 0 && row_stride % 4 == 0 && history_stride % 4 == 0 &&
+  const bool wide = hidden % 4 == 0 && base_stride % 4 == 0 && stride % 4 == 0 && row_stride % 4 == 0 && extra_stride % 4 == 0 && history_stride % 4 == 0 &&
                     keep_stride % 4 == 0 && state_stride % 4 == 0 && aligned16(base, terms, extra, gain) &&
                     aligned16(history, keep, stream, out) && aligned16(shift_share, state, out_gain, nullptr);
   const int pieces = wide ? hidden / 4 : hidden;

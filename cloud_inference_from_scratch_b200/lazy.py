@@ -113,7 +113,7 @@ class NormedUpdate:
 class WeightedTerms:
     """A weighted sum that has not been taken yet: row t is ``sum_j weights[t, j] * terms[t, j]``, with ``terms`` float32
     [T, count * H] (the ``count`` terms of a row side by side) and ``weights`` float32 [T, count] (None: all ones; then
-    ``count`` is given), plus ``extra[t]`` (float32 [T, H]) if there is one.  Whoever reads the stream next takes it in its
+    ``count`` is given), plus ``extra[t]`` (float32 [T, H], or ``Partials``) if there is one.  Whoever reads the stream next takes it in its
     own kernel, in float32, in ascending order."""
 
     def __init__(self, terms: Any, weights: Any, count: int = 0, extra: Any = None) -> None:

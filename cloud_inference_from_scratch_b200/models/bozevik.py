@@ -28,14 +28,15 @@ def _mixer(config: BozevikConfig, mixer: SharedLatentConfig) -> PartSpec:
     inner = PartSpec("latent_attention",
                      dict(hidden_size=config.width, num_heads=mixer.heads, head_dim=mixer.dim, rot_dim=mixer.rot_dim,
                           value_dim=mixer.vdim, kv_rank=mixer.kv_rank, q_rank=mixer.q_rank, scale=mixer.scale,
-                          position=position, norm_eps=config.norm_eps, shares_cache=mixer.kv_from is not None),
+                          position=position, norm_eps=config.norm_eps, shares_cache=mixer.kv_from is not None,
+                          split_output=True),
                      prefix="mix.")
     return PartSpec("token_shift", dict(hidden_size=config.width, inner=inner, name="shift"))
 
 
 def _unit(config: BozevikConfig, unit: UnitConfig, prefix: str) -> PartSpec:
     return PartSpec("clamped_glu", dict(hidden_size=config.width, intermediate_size=unit.ff, limit=unit.limit, slope=SLOPE,
-                                        shift=UP_SHIFT, bias=False), prefix=prefix)
+                                        shift=UP_SHIFT, bias=False, split_output=True), prefix=prefix)
 
 
 def _feed_forward(config: BozevikConfig, mlp: UnitFeedForwardConfig) -> PartSpec:

@@ -721,8 +721,8 @@ class Ops:
             lib = _Lib(load_library("stream_step.cu"))
             self._stream_advance = lib.function(
                 "cie_stream_advance",
-                [v, ll, v, i, ll, ll, v, v, v, f, i, v, ll, i, v, v, ll, v, v, i, v, i, i, v, v, ll, v, v, v, v, i, i, v, f,
-                 i, v, v])
+                [v, ll, v, i, ll, ll, v, v, i, ll, v, f, i, v, ll, i, v, v, ll, v, v, i, v, i, i, v, v, ll, v, v, v, v, i, i,
+                 v, f, i, v, v])
             self.stream_step_max_width = int(lib.handle.cie_stream_step_max_width())
             self._stream_step_lib = lib
 
@@ -753,12 +753,18 @@ class Ops:
         if isinstance(pending, Accumulated):
             raise KernelError("advance: an update that is already in the stream")
         extra = weights = data = None
-        terms = stride = row_stride = 0
+        terms = stride = row_stride = extras = extra_stride = 0
         if isinstance(pending, Partials) and (pending.splits == 0 or pending.bias is not None):
             pending = self.resolve(pending, self.torch.empty(pending.shape, dtype=self.torch.float32, device=self.device))
         if isinstance(pending, WeightedTerms):
             data, terms, stride, row_stride = pending.terms, pending.count, hidden, pending.count * hidden
             weights, extra = pending.weights, pending.extra
+            if isinstance(extra, Partials):
+                if extra.splits == 0 or extra.bias is not None:
+                    raise KernelError("advance: a further term that is not a plain sum")
+                extra, extras, extra_stride = extra.data, extra.splits, extra.stride
+            elif extra is not None:
+                extras = 1
         elif isinstance(pending, Partials):
             data, terms, stride, row_stride = pending.data, pending.splits, pending.stride, hidden
         elif pending is not None:
@@ -781,7 +787,7 @@ class Ops:
         self.launches += 1 if singles else 2
         request = (_ptr(ctx.query_start), _ptr(ctx.request_of_token), _ptr(ctx.slots), _ptr(ctx.request_active)) if shift is not None else (None,) * 4
         self._stream_advance(_ptr(base), base.stride(0), _ptr(data), terms, stride, row_stride, _ptr(weights), _ptr(extra),
-                             _ptr(gain), float(eps), kind, _ptr(history), history_stride, place if share is not None else 0,
+                             extras, extra_stride, _ptr(gain), float(eps), kind, _ptr(history), history_stride, place if share is not None else 0,
                              _ptr(share), keep, history_stride, _ptr(stream), _ptr(out), out_kind, _ptr(rows), count, hidden,
                              _ptr(share_vector), _ptr(state), state_stride, *request, slots, 1 if singles else 0,
                              _ptr(norm[0]) if norm is not None else None, float(norm[1]) if norm is not None else 0.0,
@@ -1078,10 +1084,11 @@ class Ops:
     # ------------------------------------------------------------------ attention over a cached latent
     def _load_latent(self) -> None:
         if self._latent_lib is None:
-            v, i, f = c_void_p, c_int, c_float
+            v, i, f, ll = c_void_p, c_int, c_float, ctypes.c_longlong
             lib = _Lib(load_library("latent.cu"))
             self._latent_prepare = lib.function(
-                "cie_latent_prepare", [v, i, v, v, v, v, v, v, i, i, v, v, v, f, i, i, i, i, i, i, i, f, i, i, v, i, v, v])
+                "cie_latent_prepare",
+                [v, i, i, ll, v, v, v, v, v, v, i, i, v, v, v, f, i, i, i, i, i, i, i, f, i, i, v, i, v, v])
             self._head_linear = lib.function("cie_head_linear", [v, i, i, v, v, i, i, v, i, i, i, i, i, i, i, v])
             self._latent_attention = lib.function(
                 "cie_latent_attention",
@@ -1104,7 +1111,8 @@ class Ops:
                 self._latent_gather = prompt.function("cie_latent_gather", [v, v, v, i, v, v, i, i, i, i, i, v, v, i, v, v])
                 self._latent_prompt = prompt.function(
                     "cie_latent_prompt",
-                    [v, i, v, i, v, i, v, v, v, i, v, i, v, v, v, v, f, i, i, i, i, i, i, i, i, f, v, v])
+                    [v, i, i, i, v, i, v, i, v, v, v, i, v, i, v, v, v, i, i, i, i, i, i, f, v, v])
+                self._latent_queries = prompt.function("cie_latent_queries", [v, i, v, v, v, f, i, i, i, i, i, i, v])
                 self._latent_prompt_lib = prompt
 
     def require_latent(self) -> int:
@@ -1171,6 +1179,14 @@ class Ops:
         self._latent_gather(_ptr(kv.k), _ptr(kv.v), _ptr(plan["portions"]), count, _ptr(blocks), _ptr(table),
                             table.shape[1], kv.num_pages, kv.page_size, rank, rot, _ptr(c_rows), _ptr(r_rows), rows,
                             _ptr(self.error_word), self.stream)
+        # the queries of the portions' tokens, which follow the step's single ones
+        first = ctx.num_single
+        tokens, padded = q.shape[0] - first, heads * (-(-dim // 16) * 16 + -(-rot // 16) * 16)
+        queries = buffer(f"latent.queries.{padded}", tokens * padded, max(tokens, self.max_rows) * padded)
+        self.launches += 1
+        self._latent_queries(_ptr(q[first:]), q.stride(0), _ptr(queries), _ptr(ctx.positions[first:]), _ptr(rotation.inv_freq),
+                             float(rotation.magnitude), int(rotation.interleaved), int(rotation.dims), tokens, heads, dim, rot,
+                             self.stream)
         width = dim + vdim
         limit = LATENT_PROMPT_BYTES // 2
         at_once = max(1, min(heads, limit // (rows * width)))
@@ -1181,16 +1197,15 @@ class Ops:
             kv_rows = expanded[: rows * part * width].view(rows, part * width)
             self.linear(c_rows, w_kv[head0 * width:(head0 + part) * width], None, kv_rows)
             self.launches += 1
-            self._latent_prompt(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(gate),
+            self._latent_prompt(_ptr(queries), tokens, heads, first, _ptr(out), out.stride(0), _ptr(gate),
                                 gate.stride(0) if gate is not None else 0, _ptr(sink), _ptr(kv_rows), _ptr(r_rows), rows,
                                 _ptr(tiles), tiles.shape[0], _ptr(ctx.context_lens), _ptr(ctx.query_lens),
-                                _ptr(ctx.query_start), _ptr(rotation.inv_freq), float(rotation.magnitude),
-                                int(rotation.interleaved), int(rotation.dims), head0, part, dim, rot, vdim, int(window),
-                                float(scale), _ptr(self.error_word), self.stream)
+                                _ptr(ctx.query_start), head0, part, dim, rot, vdim, int(window), float(scale),
+                                _ptr(self.error_word), self.stream)
 
     def latent_prepare(self, down: Any, q_out: Any, q_gain: Any, kv_gain: Any, ctx: Any, kv: Any, rotation: Any,
                        q_rank: int, rank: int, rot: int, eps: float, has_kv: bool, write_cache: bool) -> None:
-        """Per token of ``down`` (float32 [T, q_rank (+ rank + rot)]): the query latent divided by its
+        """Per token of ``down`` (float32 [T, q_rank (+ rank + rot)], or ``Partials`` of it): the query latent divided by its
         root mean square times ``q_gain`` goes to ``q_out``; with ``has_kv`` and ``write_cache`` the
         latent, normalised likewise with ``kv_gain``, and the key part, rotated by the token's position,
         go into the pages (``kv.k``: latents, ``kv.v``: rotated key parts).  ``rotation`` gives
@@ -1199,7 +1214,13 @@ class Ops:
         self._load_latent()
         table = ctx.block_tables[kv.group]
         self.launches += 1
-        self._latent_prepare(_ptr(down), down.stride(0), _ptr(q_out), _ptr(q_gain), _ptr(kv_gain), _ptr(ctx.positions),
+        terms, term_stride = 1, 0
+        if isinstance(down, Partials):
+            if down.splits == 0 or down.bias is not None:
+                raise KernelError("latent_prepare: rows that are not a plain sum")
+            terms, term_stride = down.splits, down.stride
+            down = down.data[: down.rows * down.width].view(down.rows, down.width)
+        self._latent_prepare(_ptr(down), down.stride(0), terms, term_stride, _ptr(q_out), _ptr(q_gain), _ptr(kv_gain), _ptr(ctx.positions),
                              _ptr(ctx.request_of_token), _ptr(table), table.shape[1], kv.num_pages, _ptr(kv.k),
                              _ptr(kv.v), _ptr(rotation.inv_freq), float(rotation.magnitude), int(rotation.interleaved),
                              int(rotation.dims), down.shape[0], q_rank, rank, rot, kv.page_size, float(eps),

@@ -26,6 +26,9 @@ layer of equal ``kv_rank``, ``rot_dim`` and rotation wrote (the schedule's ``rea
 ``q_rank`` 0: no query latent; ``q = W_q h`` straight from the input (tensor ``q``).  ``window`` > 0: a query at
 position i sees the keys j with 0 <= i - j < window only, and the pages behind the window are given back.
 
+``split_output``: the result may be handed on as ``Partials`` (a product of few rows cut along K), for a reader that
+adds them up.
+
 Tensor names (after the part's prefix): ``dq``, ``dq.norm``, ``uq``, ``dkv``, ``dkv.norm``, ``uk``, ``uv``,
 ``sink``, ``g``, ``o``, and ``q`` when there is no query latent; ``names`` maps them to others.
 """
@@ -44,7 +47,7 @@ class LatentAttention(Mixer):
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, value_dim: int,
                  kv_rank: int, q_rank: int, scale: float, position: PartSpec, norm_eps: float,
                  sink: bool = False, gate: bool = False, shares_cache: bool = False,
-                 names: dict[str, str] | None = None, window: int = 0) -> None:
+                 names: dict[str, str] | None = None, window: int = 0, split_output: bool = False) -> None:
         self.hidden_size = int(hidden_size)
         self.num_heads = int(num_heads)
         self.head_dim = int(head_dim)
@@ -58,6 +61,7 @@ class LatentAttention(Mixer):
         self.gate = bool(gate)
         self.shares_cache = bool(shares_cache)
         self.window = int(window)
+        self.split_output = bool(split_output)
         if self.window < 0 or self.q_rank < 0:
             raise ValueError("latent attention: window and q_rank must not be negative")
         self.position = build_part("position", position)
@@ -152,7 +156,8 @@ class LatentAttention(Mixer):
             raise ValueError("a latent-attention layer either makes its own latent or reads another layer's")
         kv = binding.kv
         down = rt.workspace.get("latent.down", tokens, self.w_down.shape[0], f32)
-        ops.linear(x, self.w_down, None, down)
+        # without a gate only latent_prepare reads these rows, and it adds partial sums up itself
+        down = ops.linear(x, self.w_down, None, down, allow_partials=bool(self.q_rank) and not self.gate, tag="latent.down")
         if self.q_rank:
             q_latent = rt.workspace.get("latent.q_latent", tokens, self.q_rank, rt.dtype)
             ops.latent_prepare(down, q_latent, self.q_gain, self.kv_gain, ctx, kv, self.rotation, self.q_rank,
@@ -182,7 +187,7 @@ class LatentAttention(Mixer):
             ops.latent_prompt(q, mixed, ctx, kv, self.rotation, plan, self.w_kv, self.sinks, heads, self.head_dim,
                               self.rot_dim, self.value_dim, self.kv_rank, self.scale, window=self.window, gate=gate)
         update = rt.workspace.get("mixer.update32", tokens, self.hidden_size, f32)
-        return ops.linear(mixed, self.w_o, None, update)
+        return ops.linear(mixed, self.w_o, None, update, allow_partials=self.split_output, tag="latent.o")
 
 
 register_part("mixer", "latent_attention", LatentAttention, replace=True)

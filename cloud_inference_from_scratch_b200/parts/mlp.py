@@ -49,17 +49,19 @@ class ClampedGLU(FeedForward):
     ``g = min(W_gate x + b_gate, limit)``, ``u = clamp(W_up x + b_up, -limit, limit)``,
     ``y = g * sigmoid(slope * g) * (u + shift)``, result ``W_down y + b_down``.  Gate and up are one
     stacked product with float32 results; biases, bounds and activation run in float32 in one kernel.
-    The result is float32 (a term of the residual sum).  Tensor names: ``gate``, ``gate.b``, ``up``,
+    The result is float32 (a term of the residual sum); ``split_output``: it may be handed on as ``Partials`` (a product
+    of few rows cut along K), for a reader that adds them up.  Tensor names: ``gate``, ``gate.b``, ``up``,
     ``up.b``, ``down``, ``down.b``."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, limit: float, slope: float = 1.702,
-                 shift: float = 1.0, bias: bool = True) -> None:
+                 shift: float = 1.0, bias: bool = True, split_output: bool = False) -> None:
         self.hidden_size = int(hidden_size)
         self.intermediate_size = int(intermediate_size)
         self.limit = float(limit)
         self.slope = float(slope)
         self.shift = float(shift)
         self.bias = bool(bias)
+        self.split_output = bool(split_output)
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         inter, hidden = self.intermediate_size, self.hidden_size
@@ -89,7 +91,7 @@ class ClampedGLU(FeedForward):
         hidden = rt.workspace.get("glu.hidden", tokens, self.intermediate_size, rt.dtype)
         rt.ops.gated_act(both, self.b_gate_up, hidden, self.slope, self.limit, self.shift)
         update = rt.workspace.get("feed_forward.update32", tokens, self.hidden_size, torch.float32)
-        return rt.ops.linear(hidden, self.w_down, self.b_down, update)
+        return rt.ops.linear(hidden, self.w_down, self.b_down, update, allow_partials=self.split_output, tag="glu.down")
 
 
 register_part("feed_forward", "clamped_glu", ClampedGLU, replace=True)

@@ -475,6 +475,7 @@ def paged(c, r, contexts, lengths, page, dtype, seed):
             v[place, :rows.stop - rows.start] = r[request][rows]
     kv = SimpleNamespace(group=0, num_pages=len(order), page_size=page, k=k.cuda(), v=v.cuda())
     ctx = step_of(lengths)
+    ctx.positions = torch.cat([torch.arange(a, a + b) for a, b in zip(contexts, lengths)]).int().cuda()
     ctx.block_tables = [table.cuda()]
     ctx.context_lens = torch.tensor(contexts, dtype=torch.int32).cuda()
     ctx.query_lens = torch.tensor(lengths, dtype=torch.int32).cuda()
