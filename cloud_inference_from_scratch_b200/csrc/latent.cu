@@ -36,7 +36,7 @@ __device__ __forceinline__ void pair_places(int i, int dims, int interleaved, in
 // only if has_kv.  The row may still be `terms` partial sums of a product cut along K, `term_stride` elements apart.
 // q_out: [T, q_rank] in the compute dtype.
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(512)
 latent_prepare_kernel(const float* __restrict__ down, int stride, int terms, size_t term_stride, T* __restrict__ q_out,
                       const float* __restrict__ q_gain, const float* __restrict__ kv_gain,
                       const int* __restrict__ positions, const int* __restrict__ request_of_token,
@@ -53,9 +53,10 @@ latent_prepare_kernel(const float* __restrict__ down, int stride, int terms, siz
   const bool keep = has_kv && write_cache && !(active && !active[request_of_token[t]]);   // not a row that only pads the batch
   const int width = q_rank + (keep ? rank + rot : 0), latent_end = q_rank + rank;
   float q_sq = 0.f, kv_sq = 0.f;
-#pragma unroll 4
+#pragma unroll 2
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
     float v = row[i];
+#pragma unroll 8
     for (int s = 1; s < terms; ++s) v += row[s * term_stride + i];
     row_s[i] = v;
     if (i < q_rank) q_sq = fmaf(v, v, q_sq);
@@ -540,7 +541,7 @@ extern "C" int cie_latent_prepare(const float* down, int stride, int terms, long
   const size_t smem = (size_t)(q_rank + (has_kv ? rank + rot : 0)) * sizeof(float);
   if (smem > 200 * 1024) CIE_FAIL("latent_prepare: a row of %zu bytes does not fit shared memory", smem);
   // few tokens: more threads a token hide the trips to memory; many: a block's reductions cost less with fewer
-  const int threads = tokens <= 148 ? 256 : 128;
+  const int threads = tokens <= 148 ? 512 : 128;
   DISPATCH_DTYPE(dtype, "latent_prepare", {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(latent_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       CIE_FAIL("latent_prepare: cannot reserve %zu bytes of shared memory", smem);

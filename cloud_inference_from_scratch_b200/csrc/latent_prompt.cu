@@ -186,7 +186,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   __shared__ float m_s[2][BM], l_s[2][BM];
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int head = a.head0 + blockIdx.y;
+  const int head = a.head0 + blockIdx.x;
   if (tid == 0) {
     for (int s = 0; s < STAGES; ++s) {
       mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1);
@@ -198,7 +198,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   }
   pdl_wait();
   pdl_trigger();
-  const int* tile = a.tiles + 4 * blockIdx.x;          // the list puts the tiles with the most keys first
+  const int* tile = a.tiles + 4 * blockIdx.y;          // the list puts the tiles with the most keys first, all heads of each
   const int request = tile[0], q0 = tile[1], row0 = tile[2], key0 = tile[3];
   const int q_len = a.query_lens[request], first_token = a.query_start[request] + q0;
   const int ntok = min(BM, q_len - q0);
@@ -217,7 +217,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   bool alive = true;
   if (warp == TMA_WARP) {
     if (lane == 0) {
-      const int column = blockIdx.y * (a.dim + a.vdim);
+      const int column = blockIdx.x * (a.dim + a.vdim);
       // the queries: plain part and rotated part begin at pieces of their own; what a piece holds beyond a part's padded
       // columns takes part in no product
       const int q_column = head * (padded16(a.dim) + padded16(a.rot)), q_row = first_token - a.token0;
@@ -472,7 +472,7 @@ extern "C" int cie_latent_prompt(const void* queries, int tokens, int all_heads,
   if (count <= 0 || heads <= 0) return 0;
   if (!cie_latent_prompt_supports(dim, rot, vdim, 8)) CIE_FAIL("latent_prompt: sizes %d + %d, %d", dim, rot, vdim);
   if (head0 < 0 || head0 + heads > all_heads) CIE_FAIL("latent_prompt: heads %d.. of %d", head0, all_heads);
-  if (rows % 128 || out_stride % 8 || heads > 65535) CIE_FAIL("latent_prompt: %d rows, stride %d, %d heads", rows, out_stride, heads);
+  if (rows % 128 || out_stride % 8 || count > 65535) CIE_FAIL("latent_prompt: %d rows, stride %d, %d tiles", rows, out_stride, count);
   if ((reinterpret_cast<uintptr_t>(kv_rows) | reinterpret_cast<uintptr_t>(r_rows) | reinterpret_cast<uintptr_t>(out) |
        reinterpret_cast<uintptr_t>(queries)) & 15)
     CIE_FAIL("latent_prompt: operands must be 16-byte aligned");
@@ -490,7 +490,7 @@ extern "C" int cie_latent_prompt(const void* queries, int tokens, int all_heads,
   }
   const PromptArgs a{(bf16*)out, out_stride, gate, gate_stride, sink, tiles, context_lens, query_lens, query_start,
                      token0, head0, dim, rot, vdim, window, scale * kLog2e, err};
-  CIE_LAUNCH("latent_prompt", latent_prompt_kernel, dim3(count, heads), dim3(THREADS), smem, (cudaStream_t)stream, q_map,
+  CIE_LAUNCH("latent_prompt", latent_prompt_kernel, dim3(heads, count), dim3(THREADS), smem, (cudaStream_t)stream, q_map,
              kv_map, r_map, a);
   return 0;
 }

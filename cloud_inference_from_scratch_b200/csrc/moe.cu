@@ -106,7 +106,7 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router,
       if (lane == 0) {
         ids[(size_t)t * top + j] = best_e;
         choice[best_e] = -FLT_MAX;
-        atomicAdd(counts + best_e, 1);
+        if (counts) atomicAdd(counts + best_e, 1);
       }
       __syncwarp();
     }
@@ -167,7 +167,7 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router,
       ids[(size_t)t * top + j] = best_e;
       weights[(size_t)t * top + j] = score[best_e];
       choice[best_e] = -FLT_MAX;
-      atomicAdd(counts + best_e, 1);
+      if (counts) atomicAdd(counts + best_e, 1);
     }
     chosen_sum += score[best_e];
     __syncwarp();
@@ -480,7 +480,7 @@ using namespace cie;
 extern "C" int cie_moe_row_tile() { return kRowTile; }
 
 // counts, offsets (experts + 1), cursors, tile_count (1) and tiles (3 * (pairs / 64 + experts)) are
-// int32 scratch of the caller; counts is zeroed here.
+// int32 scratch of the caller; counts is zeroed here.  counts null: only the choices and their weights are wanted.
 extern "C" int cie_moe_route(const void* x, const float* router, const float* correction, int* ids,
                              float* weights, int* counts, int* offsets, int* cursors, int* place_to_pair,
                              int* tiles, int* tile_count, int tokens, int hidden, int experts, int top,
@@ -495,7 +495,7 @@ extern "C" int cie_moe_route(const void* x, const float* router, const float* co
   if (experts < 1 || experts > kMaxExperts) CIE_FAIL("moe_route: 1..%d experts, got %d", kMaxExperts, experts);
   if (top < 1 || top > experts || top > 32) CIE_FAIL("moe_route: top %d of %d experts (at most 32)", top, experts);
   cudaStream_t s = (cudaStream_t)stream;
-  if (cudaMemsetAsync(counts, 0, sizeof(int) * experts, s) != cudaSuccess) CIE_FAIL("moe_route: memset failed");
+  if (counts && cudaMemsetAsync(counts, 0, sizeof(int) * experts, s) != cudaSuccess) CIE_FAIL("moe_route: memset failed");
   const int warps = kRouteWarps;
   const size_t smem = (size_t)(((2 * experts + 3) & ~3) + (hidden > groups ? hidden : groups)) * sizeof(float);
   if (smem > 200 * 1024) CIE_FAIL("moe_route: a row of %d elements does not fit shared memory", hidden);
@@ -515,6 +515,7 @@ extern "C" int cie_moe_route(const void* x, const float* router, const float* co
   } else {
     CIE_FAIL("moe_route: unknown element type code %d", dtype);
   }
+  if (!counts) return 0;
   CIE_LAUNCH("moe_plan", moe_plan_kernel, dim3(1), dim3(1024), 0, s, ids, counts, offsets, cursors, place_to_pair,
              tiles, tile_count, tokens * top, experts);
   return 0;

@@ -3,7 +3,7 @@
 from __future__ import annotations
 
 GENERIC = ("elementwise.cu", "gemm_simt.cu", "gemm_stream.cu", "gemm_tcgen05.cu", "gemm_skinny.cu", "attention_generic.cu", "sampling.cu",
-           "streams.cu", "lightning.cu", "moe.cu", "moe_tcgen05.cu", "latent.cu", "latent_tensor.cu", "latent_prompt.cu", "delta.cu", "recurrent.cu", "gla.cu",
+           "streams.cu", "lightning.cu", "moe.cu", "moe_tcgen05.cu", "moe_few.cu", "latent.cu", "latent_tensor.cu", "latent_prompt.cu", "delta.cu", "recurrent.cu", "gla.cu",
            "grouped_norm.cu", "ssd.cu", "stream_step.cu")
 
 

@@ -1405,6 +1405,12 @@ class Ops:
             self.moe_row_tile = int(lib.handle.cie_moe_row_tile())
             self._moe_lib = lib
             self._moe_tcgen05_lib = None
+            self.moe_few_pairs = 0
+            if self.code == BF16 and os.environ.get("CIE_MOE_FEW", "1") != "0":
+                few = _Lib(load_library("moe_few.cu"))
+                self._moe_gate_up_few = few.function("cie_moe_gate_up_few", [v, v, v, v, i, i, i, i, i, i, f, f, f, v, v])
+                self._moe_down_few = few.function("cie_moe_down_few", [v, v, v, v, i, i, i, i, i, v])
+                self.moe_few_pairs = int(few.handle.cie_moe_few_pairs())
 
     def _load_moe_tcgen05(self) -> None:
         if self._moe_tcgen05_lib is None:
@@ -1465,8 +1471,10 @@ class Ops:
         act = workspace.get("moe.act", tokens, top * ff, self.dtype)
         rows = workspace.get("moe.rows", tokens, top * hidden, torch.float32)
         code = self._code_of(x)
-        self.launches += 5
-        self._moe_route(_ptr(x), _ptr(router), _ptr(correction), _ptr(ids), _ptr(weights), _ptr(counts),
+        # few pairs (a decode step) stream the chosen experts' weights and need no plan
+        few = w_up is None and pairs <= self.moe_few_pairs and max(hidden, ff) <= 12288
+        self.launches += 4 if few else 5
+        self._moe_route(_ptr(x), _ptr(router), _ptr(correction), _ptr(ids), _ptr(weights), None if few else _ptr(counts),
                         _ptr(offsets), _ptr(cursors), _ptr(place_to_pair), _ptr(tiles), _ptr(tile_count), tokens,
                         hidden, experts, top, 1 if renormalize else 0, _ptr(router_bias), 1 if chosen_softmax else 0,
                         1 if sigmoid else 0, groups[0], groups[1], float(norm_floor), code, self.stream)
@@ -1475,7 +1483,11 @@ class Ops:
         aligned = (x.data_ptr() | w_gate.data_ptr() | w_down.data_ptr() | act.data_ptr()) % 16 == 0
         if w_up is None and not (code == BF16 and aligned):
             raise KernelError("routed_experts: interleaved gate/up weights are for aligned bfloat16 operands")
-        if w_up is None and os.environ.get("CIE_MOE_TCGEN05", "1") != "0":
+        if few:
+            self._moe_gate_up_few(_ptr(x), _ptr(w_gate), _ptr(act), _ptr(ids), tokens, top, experts, ff, hidden, *glu,
+                                  self.stream)
+            self._moe_down_few(_ptr(act), _ptr(w_down), _ptr(rows), _ptr(ids), tokens, top, experts, ff, hidden, self.stream)
+        elif w_up is None and os.environ.get("CIE_MOE_TCGEN05", "1") != "0":
             # tcgen05: the rows of every expert gathered side by side, tiles by TMA, accumulators in
             # tensor memory
             self._load_moe_tcgen05()
