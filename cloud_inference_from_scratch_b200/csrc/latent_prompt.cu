@@ -57,6 +57,12 @@ __device__ __forceinline__ uint32_t pack(float a, float b) {
   return *reinterpret_cast<const uint32_t*>(&pair);
 }
 
+// Behind tcgen05.wait::ld: what is done with these registers stays behind it too.
+__device__ __forceinline__ void pin(uint32_t (&r)[32]) {
+#pragma unroll
+  for (int i = 0; i < 32; ++i) asm volatile("" : "+r"(r[i]));
+}
+
 // ---------------------------------------------------------------- gather
 // portions: (request, first row, first key) of every portion, rows ascending, then (.., rows in all, ..); block_portion[b]:
 // the portion that row 128 b belongs to.  A warp a row; rows beyond the last are zeros.
@@ -301,24 +307,26 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       const int hi = pos - k0;                                           // columns lo .. hi of this tile are visible
       const int lo = a.window > 0 ? hi - a.window + 1 : 0;
       const bool masked = k0 + BN - 1 > pos_lo || (a.window > 0 && k0 < valid_hi - a.window);      // the same for the CTA
-      // the row of S comes twice, 32 columns at a time: for its maximum, and for the weights
+      // the row of S comes twice: for its maximum, and, 32 columns at a time, for the weights
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+      uint32_t raw[2][32];
+      {
+        uint32_t all[BN / 32][32];
 #pragma unroll
-      for (int c = 0; c < BN / 32; c += 2) {
-        uint32_t raw[2][32];
-        tmem_ld32(s_addr + c * 32, raw[0]);
-        tmem_ld32(s_addr + c * 32 + 32, raw[1]);
+        for (int c = 0; c < BN / 32; ++c) tmem_ld32(s_addr + c * 32, all[c]);
         tc_wait_ld();
         if (masked) {
 #pragma unroll
-          for (int i = 0; i < 64; ++i) {
-            const bool in = c * 32 + i <= hi && c * 32 + i >= lo;
-            mx4[i & 3] = fmaxf(mx4[i & 3], in ? __uint_as_float(raw[i >> 5][i & 31]) : -INFINITY);
+          for (int i = 0; i < BN; ++i) {
+            if (i > hi || i < lo) all[i >> 5][i & 31] = 0xff800000u;      // -inf: out of the maximum
+            mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(all[i >> 5][i & 31]));
           }
         } else {
 #pragma unroll
-          for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(raw[i >> 5][i & 31]));
+          for (int i = 0; i < BN; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(all[i >> 5][i & 31]));
         }
+#pragma unroll
+        for (int i = 0; i < 32; ++i) raw[0][i] = all[0][i];
       }
       const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * a.scale_log2;
       const bool grow = mx > m_used + kGrow;            // false while the row has seen no key
@@ -345,18 +353,22 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       float l4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int c = 0; c < BN / 32; ++c) {
-        uint32_t raw[32], terms[32];
-        tmem_ld32(s_addr + c * 32, raw);
-        tc_wait_ld();
-        if (masked) {
+        uint32_t terms[32];
+        uint32_t (&here)[32] = raw[c & 1];
+        if (c > 0) {
+          tc_wait_ld();
+          pin(here);
+          if (masked) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i)
-            if (c * 32 + i > hi || c * 32 + i < lo) raw[i] = 0xff800000u;      // -inf: a weight of 0
+            for (int i = 0; i < 32; ++i)
+              if (c * 32 + i > hi || c * 32 + i < lo) here[i] = 0xff800000u;      // -inf: a weight of 0
+          }
         }
+        if (c + 1 < BN / 32) tmem_ld32(s_addr + (c + 1) * 32, raw[(c + 1) & 1]);     // on its way while this one is used
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          const float p0 = fast_exp2(fmaf(__uint_as_float(raw[i]), a.scale_log2, -m_eff));
-          const float p1 = fast_exp2(fmaf(__uint_as_float(raw[i + 1]), a.scale_log2, -m_eff));
+          const float p0 = fast_exp2(fmaf(__uint_as_float(here[i]), a.scale_log2, -m_eff));
+          const float p1 = fast_exp2(fmaf(__uint_as_float(here[i + 1]), a.scale_log2, -m_eff));
           l4[(i >> 1) & 3] += p0 + p1;
           const __nv_bfloat162 first = __floats2bfloat162_rn(p0, p1);
           const float2 back = __bfloat1622float2(first);
