@@ -123,9 +123,10 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router,
     sum = warp_sum(sum);
   }
   for (int e = lane; e < experts; e += 32) {
-    const float s = sigmoid ? 1.f / (1.f + expf(-score[e])) : expf(score[e] - m) / sum;
+    const float z = score[e], s = sigmoid ? 1.f / (1.f + expf(-z)) : expf(z - m) / sum;
     score[e] = s;
-    choice[e] = s + (correction ? correction[e] : 0.f);
+    // sigmoids that nothing is added to lie in the order of their logits, which stay apart where the sigmoids round to 1
+    choice[e] = sigmoid && !correction && keep_groups == groups ? z : s + (correction ? correction[e] : 0.f);
   }
   __syncwarp();
   if (keep_groups < groups) {

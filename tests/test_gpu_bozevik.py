@@ -456,6 +456,26 @@ def test_routed_experts_with_weighted_inputs_a_clamp_and_a_shared_expert(dtype, 
         close(out, want, dtype, loose=4e-2, tight=2e-5)
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_experts_are_told_apart_where_their_scores_round_to_one(dtype):
+    from cloud_inference_from_scratch_b200.config import PartSpec
+    from cloud_inference_from_scratch_b200.parts import build_part
+
+    rt = runtime(dtype)
+    part = build_part("feed_forward", PartSpec("routed_experts", dict(
+        hidden_size=16, intermediate_size=16, num_experts=4, top=1, correction=False, score="sigmoid", defer_sum=True,
+        weight_inputs=True, activation=(9.0, 1.702, 1.0))))
+    tensors = {"router": torch.ones(4, 16) * torch.tensor([[2.0], [2.5], [3.0], [2.25]])}
+    for e in range(4):
+        for name in ("gate", "up", "down"):
+            tensors[f"e{e}.{name}"] = torch.full((16, 16), 0.01 * (e + 1)).to(rt.dtype)
+    part.bind({name: t.cuda() for name, t in tensors.items()}, rt)
+    out = torch.empty(1, 16, dtype=torch.float32).cuda()
+    rt.ops.advance(torch.zeros(1, 16).cuda(), part.forward(torch.ones(1, 16, dtype=rt.dtype).cuda(), SimpleNamespace()), out)
+    want = plain.clamped_unit(torch.ones(1, 16, dtype=F), {n: tensors["e2." + n].double() for n in ("gate", "up", "down")}, 9.0)
+    close(out, want, dtype, scale=float(want.max()), loose=2e-2)
+
+
 def paged(c, r, contexts, lengths, page, dtype, seed):
     """Pages that hold rows [c | r] (one list of rows a request), in random order, and the step's device arrays."""
     total = [a + b for a, b in zip(contexts, lengths)]
